@@ -95,7 +95,7 @@ class SequenceCache:
         by_need: dict[KVNeed, list] = {}
 
         def place(key, need):
-            # `key`: the entry's number, or (entry, part) for a part of a `MultiNeed`
+            # `key`: the entry's number, or (its key, part) for a part of a `MultiNeed`
             if isinstance(need, KVNeed):
                 by_need.setdefault(need, []).append(key)
             elif isinstance(need, StateNeed):
@@ -104,7 +104,7 @@ class SequenceCache:
                     lambda: torch.zeros(shape, dtype=_DTYPES[need.dtype], device=device),
                     f"the per-sequence state of cache entry {key}",
                     int(np.prod(shape)) * _DTYPES[need.dtype].itemsize)
-            elif isinstance(need, MultiNeed) and not isinstance(key, tuple):
+            elif isinstance(need, MultiNeed):
                 for i, part in enumerate(need.parts):
                     place((key, i), part)
             elif need is not None:

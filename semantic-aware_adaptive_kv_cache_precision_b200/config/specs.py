@@ -98,7 +98,9 @@ class AttentionSpec:
 
 @dataclass(frozen=True)
 class GatedMLPSpec:
-    """Dense gated feed-forward: `down(act(gate(x)) * up(x))`."""
+    """Dense gated feed-forward: `down(act(gate(x)) * up(x))`. `activation` "silu", or "clamped":
+    with g = min(gate(x), limit) and u = up(x) within +-limit, `down(g sigmoid(alpha g) (u +
+    plus))`."""
     hidden: int
     intermediate: int
     activation: str
@@ -106,6 +108,9 @@ class GatedMLPSpec:
     kind: str = "gated_mlp"
     #: the three tensors' names after the part's prefix: gate, up, down
     names: tuple = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
+    limit: float = float("inf")
+    alpha: float = 1.0
+    plus: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -221,10 +226,12 @@ class DifferentialAttentionSpec:
 @dataclass(frozen=True)
 class ClampedExpertSpec:
     """A gated feed-forward with clamped branches: g = min(Wgate x, limit), u = clamp(Wup x,
-    -limit, limit), y = g * sigmoid(alpha * g) * (u + 1), out = Wdown y."""
+    -limit, limit), y = g * sigmoid(alpha * g) * (u + plus), out = Wdown y. With `limit`
+    infinite, `alpha` 1 and `plus` 0 it is the plain gated one, silu(Wgate x) * (Wup x)."""
     intermediate: int
     limit: float
     alpha: float = 1.702
+    plus: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -236,7 +243,9 @@ class RoutedExpertsSpec:
     (`correction`) is added to the scores for the CHOICE only; the weights are the scores
     without it. `identity` n: the router has n more outputs after the experts'; an "expert"
     chosen among them has no tensors and returns its input (times the weight).
-    `renormalize`: whether the chosen scores are divided by their sum. `weight_input`: the
+    `groups` g: the router's outputs form g equal groups of neighbours, a group's score is the
+    largest in it, and only the outputs of the `keep_groups` best groups can be chosen.
+    `renormalize`: the chosen scores are divided by (their sum + 1e-20). `weight_input`: the
     score multiplies the expert's input (out = sum expert(w x)) rather than its output.
     `shared`: one more expert that every token uses, multiplied by `sigmoid(Wsg x)`, one
     number a token (`shared.sg`), if `shared_gate`.
@@ -254,7 +263,17 @@ class RoutedExpertsSpec:
     weight_input: bool = True
     correction: bool = False
     identity: int = 0
+    groups: int = 1
+    keep_groups: int = 1
     kind: str = "routed_experts"
+
+
+@dataclass(frozen=True)
+class QueryTemperature:
+    """Queries grow slowly with their position: at position p they are multiplied by `1 + coef *
+    ln(floor((p + 1) / every) + 1)`."""
+    coef: float
+    every: float
 
 
 @dataclass(frozen=True)
@@ -268,12 +287,16 @@ class WindowSinkAttentionSpec:
     (`window` None: every earlier key; `sink` False: the plain softmax). Kept tokens keep their
     true positions. `qk_norm` "whole": queries and keys are each divided by the root mean square
     of their WHOLE projection (all heads together, `eps` inside the root) and multiplied by a
-    weight of that size, before the rotation; None: no norm. `position`: a rotation of the first
+    weight of that size, before the rotation; "head": each head by its own root mean square,
+    without a weight; None: no norm. `q_temp`: queries are multiplied by a number of their
+    position. `gate`: the heads' outputs are multiplied element by element by `sigmoid(Wg h)`,
+    read from the mixer's input, before the output projection. `position`: a rotation of the first
     `rotary_dim` numbers of every head, or None. Values may have a width of their own; `bias`:
     q, k, v have biases. The heads' outputs are multiplied by `out_scale` before the output
     projection.
 
-    Tensor names after the part's prefix: `q`, `k`, `v` (+ `.b`), `q.norm`, `k.norm`, `sink`, `o`."""
+    Tensor names after the part's prefix: `q`, `k`, `v` (+ `.b`), `g`, `q.norm`, `k.norm`,
+    `sink`, `o`."""
     hidden: int
     heads: int
     kv_heads: int
@@ -288,6 +311,8 @@ class WindowSinkAttentionSpec:
     qk_norm: Optional[str] = "whole"
     bias: bool = True
     out_scale: float = 1.0
+    q_temp: Optional[QueryTemperature] = None
+    gate: bool = False
     kind: str = "window_sink_attention"
 
 
@@ -330,13 +355,19 @@ class DecayAttentionSpec:
 class ParallelMixerSpec:
     """Two mixers side by side that read the same input; the mixer's output is the sum of
     theirs (each already multiplied by its own `out_scale`). Both must offer the branch
-    interface (`input_decls`, `mix`, `w_o`): their input matrices are one product.
+    interface (`input_decls`, `mix`, `w_o`): their input matrices are one product. `branch_norm`:
+    each branch's output is normed over the model's width (with a weight of its own) before the
+    sum. The sum is multiplied by `scale`.
 
-    Tensor names: the branches' own, after the part's prefix + `names[i]` + "."."""
+    Tensor names: the branches' own, after the part's prefix + `names[i]` + "."; the branches'
+    norms after `names[i]` + "." + `norm_name`."""
     hidden: int
     left: object
     right: object
     names: tuple = ("left", "right")
+    branch_norm: Optional[NormSpec] = None
+    norm_name: str = "out"
+    scale: float = 1.0
     kind: str = "parallel_mixer"
 
 
@@ -360,6 +391,33 @@ class SelectiveScanSpec:
     dt_rank: int
     taps: int
     kind: str = "selective_scan"
+
+
+@dataclass(frozen=True)
+class DualScanSpec:
+    """The state-space dual mixer (Mamba-2): `[z | x | B | C | dt] = Win h` (`heads * value_dim`,
+    the same, `groups * state` twice, `heads`); x, B and C together pass a causal convolution a
+    channel over `taps` tokens with a bias (last column: the current token; zeros before the
+    start) and silu; `dt = softplus(dt + dt_bias)`; per head h, which reads B and C of group
+    floor(h / (heads / groups)),
+
+        S <- exp(-exp(A_log) dt) S + dt B x^T   (state x value_dim);   y = S^T C + D x
+
+    y is multiplied by `silu(z)`, then each of `norm_groups` equal parts of the row is divided by
+    its own root mean square (`eps` inside the root), times a weight, and projected. State a
+    sequence: S (fp32) and the convolution's last `taps - 1` inputs.
+
+    Tensor names after the part's prefix: `in`, `conv`, `conv.b`, `dt_bias`, `A_log`, `D`,
+    `norm`, `o`."""
+    hidden: int
+    heads: int
+    value_dim: int
+    state: int
+    groups: int
+    taps: int
+    norm_groups: int
+    eps: float
+    kind: str = "dual_scan"
 
 
 @dataclass(frozen=True)
@@ -456,6 +514,25 @@ class OutputNormBlockSpec:
 
 
 @dataclass(frozen=True)
+class PostNormBlockSpec:
+    """A layer whose norms come AFTER the residual sum:
+
+        x <- norm1(alpha x + mixer(x));   x <- norm2(alpha x + ffn(x))
+
+    The sublayers read the stream itself. `ffn` None: the layer has no feed-forward (and no
+    `norm2`)."""
+    prefix: str
+    mixer: object
+    ffn: object
+    norm: NormSpec
+    alpha: float
+    mixer_name: str = "mix"
+    ffn_name: str = "mlp"
+    norm_names: tuple = ("norm1", "norm2")
+    kind: str = "post_norm_block"
+
+
+@dataclass(frozen=True)
 class LayerCall:
     """One entry of the run order: run block `block` with cache entry `cache`.
 
@@ -482,7 +559,9 @@ class ModelSpec:
     `c * tanh(logits / c)` (None: neither); `head_bias_name` names a bias [vocab] of the
     output head. `ignore_tensors`: shell-style patterns of tensor names that a checkpoint
     of this architecture may hold without any part reading them (buffers that exporters
-    write, such as a rotary table's `inv_freq`); anything else unexpected is an error."""
+    write, such as a rotary table's `inv_freq`); anything else unexpected is an error.
+    `position_name` names a table [max_positions, hidden] of learned position vectors that are
+    added to the (scaled) embedding rows; None: there is none."""
     architecture: str
     vocab_size: int
     hidden: int
@@ -504,6 +583,7 @@ class ModelSpec:
     ignore_tensors: tuple = ()
     streams: int = 1
     input_mix_name: Optional[str] = None
+    position_name: Optional[str] = None
 
     def cache_entries(self) -> int:
         return 1 + max((c.cache for c in self.run_order), default=-1)

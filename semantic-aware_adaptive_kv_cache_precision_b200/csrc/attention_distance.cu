@@ -65,6 +65,10 @@ struct AttentionExtra {
   // elements of the queries' type. Null: none (or `gate_off` inside qkv).
   const void* head_gate;
   long long head_gate_stride;
+  // A gate element by element from an fp32 tensor of its own, with one map: column c of head
+  // h's output is multiplied by sigmoid(elem_gate[t * stride + h * vdim + c]). Null: none.
+  const float* elem_gate;
+  long long elem_gate_stride;
 };
 
 namespace {
@@ -656,10 +660,18 @@ distance_attention_tiled_kernel(
       gate = 1.f / (1.f + expf(-z));
     }
     const float inv = gate * x.out_scale / l[p];
+    const float* eg = x.elem_gate == nullptr
+                          ? nullptr
+                          : x.elem_gate + (long long)t * x.elem_gate_stride +
+                                (long long)(h0 + p) * vdim;
 #pragma unroll
-    for (int i = 0; i < VPL; ++i)
-      if (lane * VPL + i < vdim)
-        out[((long long)t * heads + h0 + p) * vdim + lane * VPL + i] = narrow<T>(acc[p][i] * inv);
+    for (int i = 0; i < VPL; ++i) {
+      const int col = lane * VPL + i;
+      if (col >= vdim) continue;
+      float v = acc[p][i] * inv;
+      if (eg != nullptr) v /= 1.f + expf(-eg[col]);
+      out[((long long)t * heads + h0 + p) * vdim + col] = narrow<T>(v);
+    }
   }
 }
 
@@ -878,7 +890,9 @@ SAKV_EXPORT int sakv_cached_attention(
     int window, int chunk, float lambda, float out_scale, float eps, int gate_elem_off,
     int splits, int key_splits, float* scratch, long long scratch_floats, int* tickets,
     int warp_stage, int heads_first, int keep_first, const float* sink, const void* head_gate,
-    long long head_gate_stride, cudaStream_t stream) {
+    long long head_gate_stride, const float* elem_gate, long long elem_gate_stride,
+    cudaStream_t stream) {
+  if (elem_gate != nullptr && maps != 1) return cudaErrorInvalidValue;
   if (keep_first < 0 || (keep_first > 0 && chunk > 0)) return cudaErrorInvalidValue;
   if (head_gate != nullptr && (maps != 1 || gate_off >= 0)) return cudaErrorInvalidValue;
   if (tokens < 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0 || vdim <= 0 ||
@@ -914,6 +928,8 @@ SAKV_EXPORT int sakv_cached_attention(
   x.sink = sink;
   x.head_gate = head_gate;
   x.head_gate_stride = head_gate_stride;
+  x.elem_gate = elem_gate;
+  x.elem_gate_stride = elem_gate_stride;
   const void* values = x.v_in_k ? k_cache : v_cache;
   if (dtype == SAKV_F32)
     return pick_tiled<float>(qkv, stride, gate_off, out, k_cache, values, positions, token_seq,

@@ -7,9 +7,13 @@
 
 namespace {
 
+// out[t] = table[ids[t]] * scale (+ pos_table[positions[t]]; the position's learned vector is not
+// scaled). An id or a position outside its table adds nothing.
 template <typename Table>
 __global__ void embed_kernel(const int32_t* __restrict__ ids, const Table* __restrict__ table,
-                             float* __restrict__ out, int hidden, int vocab, long long count) {
+                             float* __restrict__ out, int hidden, int vocab, long long count,
+                             float scale, const Table* __restrict__ pos_table,
+                             const int32_t* __restrict__ positions, int pos_rows) {
   let_next_kernel_start();
   wait_for_previous_kernel();
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < count;
@@ -17,7 +21,12 @@ __global__ void embed_kernel(const int32_t* __restrict__ ids, const Table* __res
     const long long token = i / hidden;
     const int col = static_cast<int>(i - token * hidden);
     const int id = ids[token];
-    out[i] = (id >= 0 && id < vocab) ? widen(table[(long long)id * hidden + col]) : 0.f;
+    float v = (id >= 0 && id < vocab) ? widen(table[(long long)id * hidden + col]) * scale : 0.f;
+    if (pos_table != nullptr) {
+      const int pos = positions[token];
+      if (pos >= 0 && pos < pos_rows) v += widen(pos_table[(long long)pos * hidden + col]);
+    }
+    out[i] = v;
   }
 }
 
@@ -144,18 +153,24 @@ SAKV_EXPORT int sakv_scale_cap(float* x, long long count, float scale, float cap
                            x, count, scale, cap);
 }
 
+// `pos_table` ([pos_rows, hidden] of the table's type, null: none): a learned vector a position,
+// added after `scale` has multiplied the token's row.
 SAKV_EXPORT int sakv_embed(const int32_t* ids, const void* table, int table_dtype, float* out,
-                           int tokens, int hidden, int vocab, cudaStream_t stream) {
-  if (tokens < 0 || hidden <= 0 || vocab <= 0) return cudaErrorInvalidValue;
+                           int tokens, int hidden, int vocab, float scale, const void* pos_table,
+                           const int32_t* positions, int pos_rows, cudaStream_t stream) {
+  if (tokens < 0 || hidden <= 0 || vocab <= 0 || (pos_table != nullptr && positions == nullptr))
+    return cudaErrorInvalidValue;
   if (tokens == 0) return 0;
   const long long count = (long long)tokens * hidden;
   const int grid = grid_for(count, 256);
   if (table_dtype == SAKV_F32)
     return launch_overlapped(embed_kernel<float>, dim3(grid), dim3(256), 0, stream, 1, ids,
-                             (const float*)table, out, hidden, vocab, count);
+                             (const float*)table, out, hidden, vocab, count, scale,
+                             (const float*)pos_table, positions, pos_rows);
   if (table_dtype == SAKV_BF16)
     return launch_overlapped(embed_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, stream, 1, ids,
-                             (const __nv_bfloat16*)table, out, hidden, vocab, count);
+                             (const __nv_bfloat16*)table, out, hidden, vocab, count, scale,
+                             (const __nv_bfloat16*)pos_table, positions, pos_rows);
   return cudaErrorInvalidValue;
 }
 

@@ -60,8 +60,18 @@ struct Params {
   __nv_bfloat16* out;
   long long ldo;
   int m_tiles, n_tiles;
+  float limit, alpha, plus;     // the clamped activation's
   int* error;
 };
+
+// silu(g) * u, or (kClamped) min(g, limit) and u within +-limit: g sigmoid(alpha g) (u + plus)
+template <bool kClamped>
+__device__ __forceinline__ float activate(const Params& p, float g, float u) {
+  if (!kClamped) return __fdividef(g, 1.0f + __expf(-g)) * u;
+  g = fminf(g, p.limit);
+  u = fminf(fmaxf(u, -p.limit), p.limit);
+  return __fdividef(g, 1.0f + __expf(-p.alpha * g)) * (u + p.plus);
+}
 
 struct Barriers {
   uint64_t full[kStages];       // (the first block's are used) both blocks' boxes have landed
@@ -71,6 +81,7 @@ struct Barriers {
   uint32_t tmem;
 };
 
+template <bool kClamped>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map,
                  const Params p) {
@@ -225,9 +236,8 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constan
           uint32_t w[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i)
-            w[i] = mma::pack_bf16(
-                __fdividef(g[2 * i], 1.0f + __expf(-g[2 * i])) * u[2 * i],
-                __fdividef(g[2 * i + 1], 1.0f + __expf(-g[2 * i + 1])) * u[2 * i + 1]);
+            w[i] = mma::pack_bf16(activate<kClamped>(p, g[2 * i], u[2 * i]),
+                                  activate<kClamped>(p, g[2 * i + 1], u[2 * i + 1]));
           if (n0 + c + 16 <= p.N) {
             *reinterpret_cast<uint4*>(dst + c) = make_uint4(w[0], w[1], w[2], w[3]);
             *reinterpret_cast<uint4*>(dst + c + 8) = make_uint4(w[4], w[5], w[6], w[7]);
@@ -260,7 +270,9 @@ int resident_pairs() {
   if (cudaGetDevice(&device) != cudaSuccess || device < 0 || device >= 64) return 0;
   if (known[device]) return known[device] - 1;
   int clusters = 0;
-  if (cudaFuncSetAttribute(gemm_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+  if (cudaFuncSetAttribute(gemm_pair_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                           kSmemBytes) == cudaSuccess &&
+      cudaFuncSetAttribute(gemm_pair_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                            kSmemBytes) == cudaSuccess) {
     cudaLaunchConfig_t config = {};
     config.gridDim = dim3(2 * sm_count());
@@ -273,7 +285,7 @@ int resident_pairs() {
     attr[0].val.clusterDim.z = 1;
     config.attrs = attr;
     config.numAttrs = 1;
-    if (cudaOccupancyMaxActiveClusters(&clusters, gemm_pair_kernel, &config) != cudaSuccess)
+    if (cudaOccupancyMaxActiveClusters(&clusters, gemm_pair_kernel<false>, &config) != cudaSuccess)
       clusters = 0;
     cudaGetLastError();
   }
@@ -299,9 +311,10 @@ SAKV_EXPORT int sakv_gemm_pair_map(void* map, const void* base, long long rows, 
 // out[M, N] (bf16, rows `ldo` apart) = silu(x Wg^T) * (x Wu^T) for W = [Wg; ...; Wu from row
 // `up_offset` on; ...] with N rows each, over tensor maps of x [M, K] and W from
 // sakv_gemm_pair_map. K, N and ldo multiples of 8, out
-// 16-byte aligned.
+// 16-byte aligned. clamped: the activation with limit, alpha and plus instead of the gated silu.
 SAKV_EXPORT int sakv_gemm_pair(const void* x_map, const void* w_map, int M, int N, int K,
-                               int up_offset, void* out, long long ldo, cudaStream_t stream) {
+                               int up_offset, void* out, long long ldo, int clamped, float limit,
+                               float alpha, float plus, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || (N % 8) || ldo < N || up_offset < N ||
       (reinterpret_cast<uintptr_t>(out) & 15) || (ldo % 8))
     return cudaErrorInvalidValue;
@@ -310,6 +323,7 @@ SAKV_EXPORT int sakv_gemm_pair(const void* x_map, const void* w_map, int M, int 
   Params p;
   p.M = M; p.N = N; p.K = K; p.up_offset = up_offset;
   p.out = reinterpret_cast<__nv_bfloat16*>(out); p.ldo = ldo; p.error = nullptr;
+  p.limit = limit; p.alpha = alpha; p.plus = plus;
   p.m_tiles = (M + 2 * BM - 1) / (2 * BM);
   p.n_tiles = (N + BN / 2 - 1) / (BN / 2);
   if (cudaGetSymbolAddress(reinterpret_cast<void**>(&p.error), g_error) != cudaSuccess)
@@ -330,7 +344,8 @@ SAKV_EXPORT int sakv_gemm_pair(const void* x_map, const void* w_map, int M, int 
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   config.attrs = attr;
   config.numAttrs = 2;
-  const cudaError_t e = cudaLaunchKernelEx(&config, gemm_pair_kernel,
+  const cudaError_t e = cudaLaunchKernelEx(&config,
+                                           clamped ? gemm_pair_kernel<true> : gemm_pair_kernel<false>,
                                            *reinterpret_cast<const CUtensorMap*>(x_map),
                                            *reinterpret_cast<const CUtensorMap*>(w_map), p);
   return e != cudaSuccess ? static_cast<int>(e) : launch_status();

@@ -15,6 +15,8 @@
 //   accumulate_f32     : R[m, n] += C                  o_proj and down_proj into the residual
 //   gated_silu         : silu(C_gate) * C_up           gate and up rows [n] and [n + I] of one
 //                                                      matrix, two accumulators side by side
+//   gated_clamped      : g sigmoid(alpha g) (u + plus) with g = min(C_gate, limit), u = C_up
+//                        within +-limit
 //
 // With few tokens and a small N there are too few row tiles to fill the GPU's SMs, so K is
 // split over the blocks of a thread-block cluster (up to 8, along blockIdx.z): every
@@ -38,7 +40,8 @@ constexpr int kThreads = 224;      // warps: 0 TMA, 1 and 6 MMA issue, 2..5 epil
 constexpr int kWTile = BM * BK * 2;
 constexpr int kMaxSplits = 8;     // portable cluster size
 
-enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_ACCUM = 2, EPI_GATED = 3 };
+enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_ACCUM = 2, EPI_GATED = 3, EPI_CLAMPED = 4 };
+constexpr bool gated_epi(int epi) { return epi == EPI_GATED || epi == EPI_CLAMPED; }
 
 struct Params {
   int M, N, K;
@@ -48,6 +51,7 @@ struct Params {
   int stages;            // tiles in flight per block (ring of shared-memory stages)
   int dual_offset;       // row of W where the "up" half starts (gated_silu)
   int epi;
+  float limit, alpha, plus;      // EPI_CLAMPED: g sigmoid(alpha g) (u + plus), g <= limit, |u| <= limit
   const void* bias;      // [N] or null
   int bias_dtype;
   void* out;             // [M, ldo]
@@ -105,6 +109,11 @@ __device__ __forceinline__ float bias_at(const Params& p, int n) {
                                   : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.bias)[n]);
 }
 
+__device__ __forceinline__ float clamped(const Params& p, float c, float up) {
+  const float g = fminf(c, p.limit), u = fminf(fmaxf(up, -p.limit), p.limit);
+  return g / (1.0f + expf(-p.alpha * g)) * (u + p.plus);
+}
+
 // (the epilogue's kind is a template argument: the choice is made once, not per element)
 template <int kEpi>
 __device__ __forceinline__ void finish(const Params& p, int part, int m, int n, float c, float up,
@@ -119,6 +128,8 @@ __device__ __forceinline__ void finish(const Params& p, int part, int m, int n, 
     // one block adds to each element exactly once, so the sum is the same every time; the
     // reduction instruction spares the thread the round trip of reading the old value
     atomicAdd(reinterpret_cast<float*>(p.out) + at, c + bias);
+  } else if (kEpi == EPI_CLAMPED) {
+    reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(clamped(p, c, up));
   } else {
     const float silu = c / (1.0f + expf(-c));
     reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(silu * up);
@@ -134,7 +145,7 @@ __device__ __forceinline__ void finish(const Params& p, int part, int m, int n, 
 template <int MT, int kEpi, int S>
 __device__ __forceinline__ void reduce_columns(const Params& p, uint32_t base, int split,
                                                int k_part, int m0, int n, int row, float bias) {
-  constexpr bool kDual = kEpi == EPI_GATED;
+  constexpr bool kDual = gated_epi(kEpi);
   constexpr int kS = S > 0 ? S : kMaxSplits;
   constexpr int kBatch = 4;
   const int splits = S > 0 ? S : p.splits;
@@ -201,6 +212,10 @@ __device__ __forceinline__ void finish4(const Params& p, int part, int m, int n,
       const float g[4] = {c.x, c.y, c.z, c.w}, u[4] = {up.x, up.y, up.z, up.w};
 #pragma unroll
       for (int i = 0; i < 4; ++i) r[i] = g[i] / (1.0f + expf(-g[i])) * u[i];
+    } else if (kEpi == EPI_CLAMPED) {
+      const float g[4] = {c.x, c.y, c.z, c.w}, u[4] = {up.x, up.y, up.z, up.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) r[i] = clamped(p, g[i], u[i]);
     }
     *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.out) + at) =
         make_uint2(mma::pack_bf16(r[0], r[1]), mma::pack_bf16(r[2], r[3]));
@@ -217,7 +232,7 @@ __device__ __forceinline__ void finish4(const Params& p, int part, int m, int n,
 template <int MT, int kEpi, int S>
 __device__ __forceinline__ void reduce_quads(const Params& p, uint32_t base, int rank, int k_part,
                                              int m0, int n0, float4 bias) {
-  constexpr bool kDual = kEpi == EPI_GATED;
+  constexpr bool kDual = gated_epi(kEpi);
   const int t = threadIdx.x - 64;                 // 0..127 among the epilogue threads
   const int r0 = (t & 31) * 4;                    // this thread's four rows (`bias`: theirs)
   const int n = n0 + r0;
@@ -259,7 +274,7 @@ template <int MT, int kEpi>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map,
                const Params p) {
-  constexpr bool kDual = kEpi == EPI_GATED;
+  constexpr bool kDual = gated_epi(kEpi);
   using C = Cfg<MT, kDual>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -476,7 +491,7 @@ __device__ int g_error;
 template <int MT, int kEpi>
 int launch(const CUtensorMap* w_map, const CUtensorMap* x_map, Params p, int n_tiles, int m_tiles,
            cudaStream_t stream) {
-  constexpr bool kDual = kEpi == EPI_GATED;
+  constexpr bool kDual = gated_epi(kEpi);
   using C = Cfg<MT, kDual>;
   static PerDeviceOnce configured;      // (attributes are per device)
   if (configured.needs()) {
@@ -523,8 +538,8 @@ SAKV_EXPORT int sakv_gemm_tc_map(void* map, const void* base, long long rows, lo
 SAKV_EXPORT int sakv_gemm_tc(const void* w_map, const void* x_map, int M, int N, int K, int mt,
                              int splits, int parts, int epi, int dual_offset, const void* bias,
                              int bias_dtype, void* out, long long ldo, long long part_stride,
-                             cudaStream_t stream) {
-  if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || splits < 1 || epi < 0 || epi > EPI_GATED ||
+                             float limit, float alpha, float plus, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || splits < 1 || epi < 0 || epi > EPI_CLAMPED ||
       ldo < N || parts < 1 || parts > 64 || (parts > 1 && epi != EPI_F32))
     return cudaErrorInvalidValue;
   const int total_kb = (K + BK - 1) / BK;
@@ -544,17 +559,19 @@ SAKV_EXPORT int sakv_gemm_tc(const void* w_map, const void* x_map, int M, int N,
   else
     p.splits = splits;
   p.dual_offset = dual_offset;
+  p.limit = limit; p.alpha = alpha; p.plus = plus;
   p.epi = epi; p.bias = bias; p.bias_dtype = bias_dtype;
   p.out = out; p.ldo = ldo; p.error = nullptr;
   const int n_tiles = (N + BM - 1) / BM;
   const int m_tiles = (M + mt - 1) / mt;
   if (m_tiles > 65535) return cudaErrorInvalidValue;
-  const bool dual = epi == EPI_GATED;
+  const bool dual = gated_epi(epi);
   const CUtensorMap* wm = (const CUtensorMap*)w_map;
   const CUtensorMap* xm = (const CUtensorMap*)x_map;
 #define GO(MT_)                                                                   \
   if (mt == MT_)                                                                  \
-    return dual ? launch<MT_, EPI_GATED>(wm, xm, p, n_tiles, m_tiles, stream)     \
+    return epi == EPI_CLAMPED ? launch<MT_, EPI_CLAMPED>(wm, xm, p, n_tiles, m_tiles, stream)     \
+         : dual ? launch<MT_, EPI_GATED>(wm, xm, p, n_tiles, m_tiles, stream)     \
          : epi == EPI_BF16 ? launch<MT_, EPI_BF16>(wm, xm, p, n_tiles, m_tiles, stream)   \
          : epi == EPI_F32 ? launch<MT_, EPI_F32>(wm, xm, p, n_tiles, m_tiles, stream)     \
                           : launch<MT_, EPI_ACCUM>(wm, xm, p, n_tiles, m_tiles, stream)

@@ -3,7 +3,9 @@
 //   route    a warp a token: the `top` largest router scores (ties: the lowest index), the
 //            scores as weights, and the token's place among the rows of each chosen expert.
 //            A score is the sigmoid of the logit, or the softmax over all the router's
-//            outputs; a bias an output may be added for the choice only. Outputs beyond the
+//            outputs; a bias an output may be added for the choice only. The outputs may form
+//            groups of neighbours of which only the best few (by their largest score) are open
+//            to a token's choice, and the chosen scores may be divided by their sum. Outputs beyond the
 //            experts that have weights are identity experts: they take no rows, and combine
 //            adds the token's own input times the weight for them
 //   plan     one block: where each expert's rows begin and which (expert, first row) every
@@ -13,7 +15,8 @@
 //            expert's INPUT) rounded once to the activations' type
 //   products out = rows x W[e]^T for every tile, with the weights of the tile's expert:
 //            the gated pair with the clamped activation in its epilogue
-//              g = min(., limit), u = clamp(., -limit, limit), y = g * sigmoid(alpha g) * (u + 1)
+//              g = min(., limit), u = clamp(., -limit, limit), y = g * sigmoid(alpha g) * (u + plus)
+//            (limit infinite, alpha 1, plus 0: the plain gated silu)
 //            and the plain product that leaves fp32
 //   combine  a token's rows summed in the order of its choices, plus the shared expert's
 //            output times sigmoid of its gate's logit
@@ -51,13 +54,24 @@ __global__ void logits_kernel(const T* __restrict__ h, const float* __restrict__
 
 // `experts`: the router's outputs; the first `real` of them have weights. softmax 0: the score
 // is sigmoid(z); 1: exp(z - max) / sum over all outputs. bias (null: none): added to the score
-// for the choice. Without a bias the sigmoid's order is the logits' own, and they are compared.
+// for the choice. Without a bias the scores' order is the logits' own, and they are compared.
+// groups > 1: the outputs form that many equal groups of neighbours; the `keep` groups with the
+// largest best score (of the choice) are open, the rest closed (ties: the lowest index).
+// renorm: the weights are the chosen scores over (their sum + 1e-20).
+struct RouteForm {
+  int softmax;
+  const float* bias;
+  int groups, keep;            // groups <= 64
+  int renorm;
+};
+
 __device__ __forceinline__ void route_token(const float* __restrict__ z, int experts, int top,
                                             int32_t* __restrict__ chosen,
                                             float* __restrict__ weights,
                                             int32_t* counts, int32_t* __restrict__ rank,
-                                            int real, int softmax,
-                                            const float* __restrict__ bias, int lane) {
+                                            int real, const RouteForm& form, int lane) {
+  const int softmax = form.softmax;
+  const float* __restrict__ bias = form.bias;
   float top_z = -INFINITY, total = 1.f;
   if (softmax) {
     for (int e = lane; e < experts; e += 32) top_z = fmaxf(top_z, z[e]);
@@ -69,14 +83,45 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int exp
   auto score = [&](float logit) {
     return softmax ? expf(logit - top_z) / total : 1.f / (1.f + expf(-logit));
   };
-  const bool by_logit = !softmax && bias == nullptr;
+  const bool by_logit = bias == nullptr;
+  auto rank_of = [&](int e) { return by_logit ? z[e] : score(z[e]) + bias[e]; };
+  const int per_group = experts / form.groups;
+  uint64_t open = ~0ull;                           // bit g: group g may be chosen from
+  if (form.groups > 1) {
+    open = 0;
+    for (int k = 0; k < form.keep; ++k) {
+      float best = -INFINITY;
+      int at = 0x7fffffff;
+      for (int g = lane; g < form.groups; g += 32) {
+        if (open >> g & 1) continue;
+        float v = -INFINITY;
+        for (int e = g * per_group; e < (g + 1) * per_group; ++e) v = fmaxf(v, rank_of(e));
+        if (v > best || at == 0x7fffffff) {
+          best = v;
+          at = g;
+        }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ob > best || (ob == best && oa < at)) {
+          best = ob;
+          at = oa;
+        }
+      }
+      open |= 1ull << (at & 63);
+    }
+  }
+  float sum_chosen = 0.f;
   uint32_t taken = 0;                              // bit i: this lane's i-th expert is chosen
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int at = 0x7fffffff;
     for (int i = 0, e = lane; e < experts; ++i, e += 32) {
       if (taken >> i & 1) continue;
-      const float v = by_logit ? z[e] : score(z[e]) + (bias ? bias[e] : 0.f);
+      if (form.groups > 1 && !(open >> (e / per_group) & 1)) continue;
+      const float v = rank_of(e);
       if (v > best || (at == 0x7fffffff && !(v != v))) {
         best = v;
         at = e;
@@ -96,19 +141,22 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int exp
     if (lane == 0) {
       chosen[k] = at;
       weights[k] = score(z[at]);
+      sum_chosen += weights[k];
       rank[k] = at < real ? atomicAdd(counts + at, 1) : -1;
     }
   }
+  if (form.renorm && lane == 0)
+    for (int k = 0; k < top; ++k) weights[k] /= sum_chosen + 1e-20f;
 }
 
 __global__ void route_kernel(const float* __restrict__ logits, long long ld, int experts, int top,
                              int32_t* __restrict__ chosen, float* __restrict__ weights,
                              int32_t* __restrict__ counts, int32_t* __restrict__ rank,
-                             int tokens, int real, int softmax, const float* __restrict__ bias) {
+                             int tokens, int real, const RouteForm form) {
   const long long t = (blockIdx.x * (long long)blockDim.x + threadIdx.x) >> 5;
   if (t >= tokens) return;
   route_token(logits + t * ld, experts, top, chosen + t * top, weights + t * top, counts,
-              rank + t * top, real, softmax, bias, threadIdx.x & 31);
+              rank + t * top, real, form, threadIdx.x & 31);
 }
 
 // Where each expert's rows begin and the tiles of the grouped products, from the experts'
@@ -146,8 +194,8 @@ __device__ __forceinline__ void plan_tiles(const int32_t* counts, int32_t* __res
 __global__ void __launch_bounds__(256)
 route_plan_kernel(const float* __restrict__ logits, long long ld, int experts, int top,
                   int32_t* __restrict__ chosen, float* __restrict__ weights,
-                  int32_t* __restrict__ rank, int tokens, int real, int softmax,
-                  const float* __restrict__ bias, int32_t* __restrict__ offsets,
+                  int32_t* __restrict__ rank, int tokens, int real, const RouteForm form,
+                  int32_t* __restrict__ offsets,
                   int32_t* __restrict__ tile_expert, int32_t* __restrict__ tile_row,
                   int32_t* __restrict__ n_tiles, int max_tiles) {
   extern __shared__ int32_t shared_ints[];         // counts [real], then base [real + 1]
@@ -156,8 +204,8 @@ route_plan_kernel(const float* __restrict__ logits, long long ld, int experts, i
   __syncthreads();
   for (int t = threadIdx.x >> 5; t < tokens; t += blockDim.x >> 5)
     route_token(logits + t * ld, experts, top, chosen + (long long)t * top,
-                weights + (long long)t * top, counts, rank + (long long)t * top, real, softmax,
-                bias, threadIdx.x & 31);
+                weights + (long long)t * top, counts, rank + (long long)t * top, real, form,
+                threadIdx.x & 31);
   __syncthreads();
   plan_tiles(counts, offsets, tile_expert, tile_row, n_tiles, real, max_tiles, counts + real);
 }
@@ -200,7 +248,7 @@ grouped_kernel(const T* __restrict__ a, const T* __restrict__ w0, const T* __res
                long long expert_stride, const int32_t* __restrict__ tile_expert,
                const int32_t* __restrict__ tile_row, const int32_t* __restrict__ offsets,
                const int32_t* __restrict__ n_tiles, void* __restrict__ out_v, int n, int k,
-               float limit, float alpha) {
+               float limit, float alpha, float plus) {
   __shared__ float as[TK][TM + 4];
   __shared__ float ws[DUAL ? 2 : 1][TK][TN + 4];
   if ((int)blockIdx.x >= *n_tiles) return;
@@ -250,7 +298,7 @@ grouped_kernel(const T* __restrict__ a, const T* __restrict__ w0, const T* __res
       if constexpr (DUAL) {
         const float g = fminf(acc[0][i][j], limit);
         const float u = fminf(fmaxf(acc[1][i][j], -limit), limit);
-        const float y = g / (1.f + expf(-alpha * g)) * (u + 1.f);
+        const float y = g / (1.f + expf(-alpha * g)) * (u + plus);
         static_cast<T*>(out_v)[(long long)row * n + col] = narrow<T>(y);
       } else {
         static_cast<float*>(out_v)[(long long)row * n + col] = acc[0][i][j];
@@ -279,7 +327,7 @@ grouped_tc_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __re
                   const __nv_bfloat16* __restrict__ w1, long long expert_stride,
                   const int32_t* __restrict__ tile_expert, const int32_t* __restrict__ tile_row,
                   const int32_t* __restrict__ offsets, const int32_t* __restrict__ n_tiles,
-                  void* __restrict__ out_v, int n, int k, float limit, float alpha) {
+                  void* __restrict__ out_v, int n, int k, float limit, float alpha, float plus) {
   constexpr int kW = DUAL ? 2 : 1;
   constexpr int kStages = DUAL ? 3 : 4;          // (48 KB of static shared memory at most)
   __shared__ __align__(16) __nv_bfloat16 as[kStages][TM][kPad];
@@ -362,7 +410,7 @@ grouped_tc_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __re
           const float g = fminf(acc[0][mt][nt][f], limit);
           const float u = fminf(fmaxf(acc[1][mt][nt][f], -limit), limit);
           static_cast<__nv_bfloat16*>(out_v)[(long long)row * n + col] =
-              __float2bfloat16_rn(g / (1.f + expf(-alpha * g)) * (u + 1.f));
+              __float2bfloat16_rn(g / (1.f + expf(-alpha * g)) * (u + plus));
         } else {
           static_cast<float*>(out_v)[(long long)row * n + col] = acc[0][mt][nt][f];
         }
@@ -372,14 +420,15 @@ grouped_tc_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __re
 // The dense form of the same activation for the shared expert: gate_up [T, 2 ff] -> [T, ff].
 template <typename T>
 __global__ void clamped_act_kernel(const T* __restrict__ gate_up, T* __restrict__ out,
-                                   long long count, int ff, float limit, float alpha) {
+                                   long long count, int ff, float limit, float alpha,
+                                   float plus) {
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < count;
        i += (long long)gridDim.x * blockDim.x) {
     const long long t = i / ff;
     const int c = static_cast<int>(i - t * ff);
     const float g = fminf(widen(gate_up[t * 2 * ff + c]), limit);
     const float u = fminf(fmaxf(widen(gate_up[t * 2 * ff + ff + c]), -limit), limit);
-    out[i] = narrow<T>(g / (1.f + expf(-alpha * g)) * (u + 1.f));
+    out[i] = narrow<T>(g / (1.f + expf(-alpha * g)) * (u + plus));
   }
 }
 
@@ -415,37 +464,46 @@ __global__ void combine_kernel(const float* __restrict__ rows, const int32_t* __
 
 SAKV_EXPORT int sakv_moe_tile_rows() { return TM; }
 
+static bool form_fits(int experts, int top, int groups, int keep) {
+  return groups >= 1 && groups <= 64 && experts % groups == 0 && keep >= 1 && keep <= groups &&
+         (long long)experts / groups * keep >= top;
+}
+
 // logits: fp32 [tokens, ld] (the first `experts` columns, of which the first `real` belong to
 // experts with weights and the rest to identity experts); counts: int32 [real], zero on entry
 // (plan leaves it zero again). chosen, rank: int32 [tokens, top] (rank -1: an identity
-// expert); weights: fp32. softmax: the score's kind; bias: fp32 [experts] or null.
+// expert); weights: fp32. softmax: the score's kind; bias: fp32 [experts] or null; groups, keep,
+// renorm: see `RouteForm`.
 SAKV_EXPORT int sakv_moe_route(const float* logits, long long ld, int experts, int top,
                                int32_t* chosen, float* weights, int32_t* counts, int32_t* rank,
-                               int tokens, int real, int softmax, const float* bias,
-                               cudaStream_t stream) {
+                               int tokens, int real, int softmax, const float* bias, int groups,
+                               int keep, int renorm, cudaStream_t stream) {
   if (tokens < 0 || experts <= 0 || experts > 1024 || top <= 0 || top > experts || top > 32 ||
-      ld < experts || real < 0 || real > experts)
+      ld < experts || real < 0 || real > experts || !form_fits(experts, top, groups, keep))
     return cudaErrorInvalidValue;
   if (tokens == 0) return 0;
   const int threads = 128;
   const long long blocks = ((long long)tokens * 32 + threads - 1) / threads;
   return launch_ordered(route_kernel, dim3((unsigned)blocks), dim3(threads), 0, stream, logits, ld,
-                        experts, top, chosen, weights, counts, rank, tokens, real, softmax, bias);
+                        experts, top, chosen, weights, counts, rank, tokens, real,
+                        RouteForm{softmax, bias, groups, keep, renorm});
 }
 
 // `sakv_moe_route` and `sakv_moe_plan` in one launch of one block, for steps of few tokens
 // (the rows' counts live in shared memory: no `counts` argument).
 SAKV_EXPORT int sakv_moe_route_plan(const float* logits, long long ld, int experts, int top,
                                     int32_t* chosen, float* weights, int32_t* rank, int tokens,
-                                    int real, int softmax, const float* bias, int32_t* offsets,
+                                    int real, int softmax, const float* bias, int groups,
+                                    int keep, int renorm, int32_t* offsets,
                                     int32_t* tile_expert, int32_t* tile_row, int32_t* n_tiles,
                                     int max_tiles, cudaStream_t stream) {
   if (tokens <= 0 || experts <= 0 || experts > 1024 || top <= 0 || top > experts || top > 32 ||
-      ld < experts || real <= 0 || real > experts || max_tiles <= 0)
+      ld < experts || real <= 0 || real > experts || max_tiles <= 0 ||
+      !form_fits(experts, top, groups, keep))
     return cudaErrorInvalidValue;
   return launch_ordered(route_plan_kernel, dim3(1), dim3(256), (size_t)(2 * real + 1) * 4, stream,
-                        logits, ld, experts, top, chosen, weights, rank, tokens, real, softmax,
-                        bias, offsets, tile_expert, tile_row, n_tiles, max_tiles);
+                        logits, ld, experts, top, chosen, weights, rank, tokens, real,
+                        RouteForm{softmax, bias, groups, keep, renorm}, offsets, tile_expert, tile_row, n_tiles, max_tiles);
 }
 
 // out[t, o] = sum_i h[t, i] w[o, i] in fp32: h [tokens, width] of `dtype`, w fp32 [outputs,
@@ -499,14 +557,15 @@ SAKV_EXPORT int sakv_moe_product(const void* a, int dtype, const void* w0, const
                                  long long expert_stride, const int32_t* tile_expert,
                                  const int32_t* tile_row, const int32_t* offsets,
                                  const int32_t* n_tiles, int max_tiles, void* out, int n, int k,
-                                 int dual, float limit, float alpha, cudaStream_t stream) {
+                                 int dual, float limit, float alpha, float plus,
+                                 cudaStream_t stream) {
   if (max_tiles <= 0 || n <= 0 || k <= 0 || (dual && !w1)) return cudaErrorInvalidValue;
   const dim3 grid(max_tiles, (n + TN - 1) / TN), block(256);
   if (grid.y > 65535) return cudaErrorInvalidValue;
 #define SAKV_GROUPED(T, DUAL)                                                                    \
   return launch_ordered(grouped_kernel<T, DUAL>, grid, block, 0, stream, (const T*)a,          \
                         (const T*)w0, (const T*)w1, expert_stride, tile_expert, tile_row,        \
-                        offsets, n_tiles, out, n, k, limit, alpha)
+                        offsets, n_tiles, out, n, k, limit, alpha, plus)
   if (dtype == SAKV_F32) {
     if (dual) SAKV_GROUPED(float, true);
     SAKV_GROUPED(float, false);
@@ -520,11 +579,11 @@ SAKV_EXPORT int sakv_moe_product(const void* a, int dtype, const void* w0, const
         return launch_ordered(grouped_tc_kernel<true>, grid, threads, 0, stream,
                               (const __nv_bfloat16*)a, (const __nv_bfloat16*)w0,
                               (const __nv_bfloat16*)w1, expert_stride, tile_expert, tile_row,
-                              offsets, n_tiles, out, n, k, limit, alpha);
+                              offsets, n_tiles, out, n, k, limit, alpha, plus);
       return launch_ordered(grouped_tc_kernel<false>, grid, threads, 0, stream,
                             (const __nv_bfloat16*)a, (const __nv_bfloat16*)w0,
                             (const __nv_bfloat16*)w1, expert_stride, tile_expert, tile_row,
-                            offsets, n_tiles, out, n, k, limit, alpha);
+                            offsets, n_tiles, out, n, k, limit, alpha, plus);
     }
     if (dual) SAKV_GROUPED(__nv_bfloat16, true);
     SAKV_GROUPED(__nv_bfloat16, false);
@@ -534,18 +593,18 @@ SAKV_EXPORT int sakv_moe_product(const void* a, int dtype, const void* w0, const
 }
 
 SAKV_EXPORT int sakv_clamped_act(const void* gate_up, void* out, int dtype, int tokens, int ff,
-                                 float limit, float alpha, cudaStream_t stream) {
+                                 float limit, float alpha, float plus, cudaStream_t stream) {
   if (tokens < 0 || ff <= 0) return cudaErrorInvalidValue;
   if (tokens == 0) return 0;
   const long long count = (long long)tokens * ff;
   const dim3 grid(grid_for(count, 256)), block(256);
   if (dtype == SAKV_F32)
     return launch_ordered(clamped_act_kernel<float>, grid, block, 0, stream, (const float*)gate_up,
-                          (float*)out, count, ff, limit, alpha);
+                          (float*)out, count, ff, limit, alpha, plus);
   if (dtype == SAKV_BF16)
     return launch_ordered(clamped_act_kernel<__nv_bfloat16>, grid, block, 0, stream,
                           (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, count, ff, limit,
-                          alpha);
+                          alpha, plus);
   return cudaErrorInvalidValue;
 }
 

@@ -7,7 +7,12 @@
 //     inputs as state, the step size dt = softplus(Wdt low + b), the gate y * silu(z);
 //   * attention without softmax whose state, a matrix a head, fades by a fixed factor a head:
 //               S <- decay_h S + k v^T;   o = S^T q          (q, k, v after silu)
-//     and the norm over all heads' outputs with its sigmoid gate.
+//     and the norm over all heads' outputs with its sigmoid gate;
+//   * the state-space dual form, a matrix a head whose decay and step the token chooses, one
+//     number a head:
+//               S <- exp(dt_h A_h) S + dt_h B x^T;   y = S^T C + D_h x,   dt_h = softplus(. + b_h)
+//     with B and C shared by the heads of a group, and the gate y * silu(z) before a norm over
+//     equal parts of the row.
 //
 // Everything that enters a recurrence is fp32: decays, exponentials, softplus, step sizes, the
 // states and the sums over them. The projections' outputs come as fp32 (their accumulators,
@@ -469,18 +474,193 @@ __global__ void decay_carry_kernel(const float* __restrict__ decay_less_one,
   if (keep_state) *home = s;
 }
 
+// ---------------------------------------------------------------------------------------
+// The state-space dual form. As in the fading state a block owns `cols` neighbouring value
+// columns of one head of one sequence and a column's `dim` rows are dealt to RS neighbouring
+// lanes, RP each; what differs is where the rows come from (B for k, C for q, both of the head's
+// group and of the convolution's output type; x for v), the step size dt a (token, head), made
+// here from the projection's column, which multiplies x and chooses the token's decay, and D x
+// added to the output. State in memory: [slots, heads, vdim, dim] (a column's rows together).
+// PHASE as above; a run's decay to the carry kernel is the sum of its step sizes.
+// ---------------------------------------------------------------------------------------
+template <typename C>
+struct DualScan {
+  const C* xbc;                    // [tokens, stride]: x, B and C after the convolution
+  long long stride;
+  int x_off, b_off, c_off;
+  const float* dt;                 // [tokens, dt_stride]: the heads' step sizes before the bias
+  long long dt_stride;
+  const float* dt_bias;            // [heads]
+  const float* a;                  // [heads], negative
+  const float* d_skip;             // [heads]
+  float* state;
+  const int32_t* cu_seqlens;
+  const int32_t* slots;
+  float* out;                      // [tokens, heads * vdim]
+  int heads, groups, dim, vdim, rs, cols, keep_state, chunk_len, max_chunks;
+  float* scratch;                  // [sequences, max_chunks, heads, vdim, dim]
+  float* dt_sums;                  // [sequences, max_chunks, heads]
+};
+
+template <int RP, int PHASE, typename C>
+__global__ void dual_scan_kernel(const DualScan<C> p) {
+  extern __shared__ __align__(16) float shared[];
+  const int padded = p.rs * RP;                     // dim rounded up to whole lanes
+  const int padded_shift = 31 - __clz(padded);
+  float* qs = shared;                               // [kRun, padded]  C
+  float* ks = qs + kRun * padded;                   // [kRun, padded]  B
+  float* vs = ks + kRun * padded;                   // [kRun, cols]    x
+  float* steps = vs + kRun * p.cols;                // [kRun]          dt
+  float* fades = steps + kRun;                      // [kRun]          exp(dt A) - 1
+  const int b = PHASE == 0 ? blockIdx.z : blockIdx.z / p.max_chunks;
+  const int piece = PHASE == 0 ? 0 : blockIdx.z % p.max_chunks;
+  int first = p.cu_seqlens[b], last = p.cu_seqlens[b + 1];
+  if (PHASE != 0) {
+    first += piece * p.chunk_len;
+    if (first >= last) return;                      // (the whole block)
+    if (last - first > p.chunk_len) last = first + p.chunk_len;
+  }
+  const int h = blockIdx.y, col0 = blockIdx.x * p.cols;
+  const int group_off = h / (p.heads / p.groups) * p.dim;
+  const int r = threadIdx.x % p.rs, j = threadIdx.x / p.rs;
+  const int col = col0 + j, dim = p.dim;
+  const bool live = col < p.vdim;
+  const float a = p.a[h], bias = p.dt_bias[h], skip = p.d_skip[h];
+  float s[RP];
+  const long long per_seq = (long long)p.heads * p.vdim * dim;
+  const long long place = ((long long)h * p.vdim + (live ? col : 0)) * dim + r * RP;
+  float* mine = PHASE == 0 ? p.state + p.slots[b] * per_seq + place
+                           : p.scratch + ((long long)b * p.max_chunks + piece) * per_seq + place;
+  const bool wide = dim % 4 == 0;                   // (then every lane's rows are 16-byte aligned)
+#pragma unroll
+  for (int k = 0; k < RP; k += 4) {
+    const int at = r * RP + k;
+    if (PHASE != 1 && live && wide && at < dim) {
+      const float4 v = *reinterpret_cast<const float4*>(mine + k);
+      s[k] = v.x; s[k + 1] = v.y; s[k + 2] = v.z; s[k + 3] = v.w;
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        s[k + i] = (PHASE != 1 && live && at + i < dim) ? mine[k + i] : 0.f;
+    }
+  }
+  float dt_sum = 0.f;
+  for (int t0 = first; t0 < last; t0 += kRun) {
+    const int run = last - t0 < kRun ? last - t0 : kRun;
+    __syncthreads();
+    if ((int)threadIdx.x < run) {
+      const float dt = softplus(p.dt[(long long)(t0 + threadIdx.x) * p.dt_stride + h] + bias);
+      steps[threadIdx.x] = dt;
+      fades[threadIdx.x] = exp_less_one<sizeof(C) == 4>(dt * a);
+    }
+    for (int e = threadIdx.x; e < run * padded; e += blockDim.x) {
+      const int tt = e >> padded_shift, i = e & (padded - 1);     // (padded is a power of two)
+      const C* row = p.xbc + (long long)(t0 + tt) * p.stride + group_off;
+      if (PHASE != 1) qs[e] = i < dim ? widen(row[p.c_off + i]) : 0.f;
+      ks[e] = i < dim ? widen(row[p.b_off + i]) : 0.f;
+    }
+    for (int e = threadIdx.x; e < run * p.cols; e += blockDim.x) {
+      const int tt = e / p.cols, i = e - tt * p.cols;
+      vs[e] = col0 + i < p.vdim ? widen(p.xbc[(long long)(t0 + tt) * p.stride + p.x_off +
+                                              (long long)h * p.vdim + col0 + i])
+                                : 0.f;
+    }
+    __syncthreads();
+    for (int tt = 0; tt < run; ++tt) {
+      const float x = vs[tt * p.cols + j], dt = steps[tt], fade = fades[tt];
+      const float v = dt * x;
+      dt_sum += dt;
+      float o = 0.f;
+      const float4* k4 = reinterpret_cast<const float4*>(ks + tt * padded + r * RP);
+      const float4* q4 = reinterpret_cast<const float4*>(qs + tt * padded + r * RP);
+#pragma unroll
+      for (int k = 0; k < RP; k += 4) {
+        const float4 kk = k4[k >> 2];
+        // S + (e^(dt A) - 1) S + dt B x: a decay close to 1 keeps its distance from 1
+        s[k] = fmaf(kk.x, v, fmaf(fade, s[k], s[k]));
+        s[k + 1] = fmaf(kk.y, v, fmaf(fade, s[k + 1], s[k + 1]));
+        s[k + 2] = fmaf(kk.z, v, fmaf(fade, s[k + 2], s[k + 2]));
+        s[k + 3] = fmaf(kk.w, v, fmaf(fade, s[k + 3], s[k + 3]));
+        if (PHASE != 1) {
+          const float4 qq = q4[k >> 2];
+          o = fmaf(s[k], qq.x, o);
+          o = fmaf(s[k + 1], qq.y, o);
+          o = fmaf(s[k + 2], qq.z, o);
+          o = fmaf(s[k + 3], qq.w, o);
+        }
+      }
+      if (PHASE != 1) {
+        for (int d = p.rs >> 1; d > 0; d >>= 1) o += __shfl_xor_sync(0xffffffffu, o, d);
+        if (r == 0 && live)
+          p.out[((long long)(t0 + tt) * p.heads + h) * p.vdim + col] = fmaf(skip, x, o);
+      }
+    }
+  }
+  if (live && (PHASE == 1 || (PHASE == 0 && p.keep_state))) {
+#pragma unroll
+    for (int k = 0; k < RP; k += 4) {
+      const int at = r * RP + k;
+      if (wide && at < dim) {
+        *reinterpret_cast<float4*>(mine + k) = make_float4(s[k], s[k + 1], s[k + 2], s[k + 3]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (at + i < dim) mine[k + i] = s[k + i];
+      }
+    }
+  }
+  if (PHASE == 1 && blockIdx.x == 0 && threadIdx.x == 0)
+    p.dt_sums[((long long)b * p.max_chunks + piece) * p.heads + h] = dt_sum;
+}
+
+// Between the two passes over a prompt's runs: one thread a (sequence, head, column, row).
+__global__ void dual_carry_kernel(const float* __restrict__ a, float* __restrict__ state,
+                                  float* __restrict__ scratch, const float* __restrict__ dt_sums,
+                                  const int32_t* __restrict__ cu_seqlens,
+                                  const int32_t* __restrict__ slots, int sequences, int heads,
+                                  long long per_head, int chunk_len, int max_chunks,
+                                  int keep_state) {
+  const long long idx = blockIdx.x * (long long)blockDim.x + threadIdx.x;
+  const long long per = heads * per_head;
+  if (idx >= sequences * per) return;
+  const int b = static_cast<int>(idx / per);
+  const long long e = idx - b * per;
+  const int h = static_cast<int>(e / per_head);
+  const int runs = (cu_seqlens[b + 1] - cu_seqlens[b] + chunk_len - 1) / chunk_len;
+  float* home = state + (long long)slots[b] * per + e;
+  float s = *home;
+  for (int j = 0; j < runs; ++j) {
+    float* p = scratch + ((long long)b * max_chunks + j) * per + e;
+    const float left = *p;
+    *p = s;
+    s += fmaf(expm1f(a[h] * dt_sums[((long long)b * max_chunks + j) * heads + h]), s, left);
+  }
+  if (keep_state) *home = s;
+}
+
 // out[t] = y[t] / sqrt(mean(y[t]^2) + eps) * w * sigmoid(gate[t]) * scale. A block a token.
 // `group` == width: the mean over the whole row (all heads' outputs together); smaller: over
 // each run of `group` numbers (a head's outputs), a warp a run. `w` null: no weight.
-// `gate_silu`: the gate is `g * sigmoid(g)` instead of `sigmoid(g)`.
+// `gate_silu`: the gate is `g * sigmoid(g)` instead of `sigmoid(g)`. `gate_first`: the gate
+// multiplies y before the mean is taken (the gated row is kept in shared memory).
 template <typename W, typename C>
 __global__ void __launch_bounds__(256)
 norm_gate_kernel(const float* __restrict__ y, const W* __restrict__ w,
                  const float* __restrict__ gate, long long gate_stride, C* __restrict__ out,
-                 int width, int group, int gate_silu, float eps, float scale) {
+                 int width, int group, int gate_silu, int gate_first, float eps, float scale) {
+  extern __shared__ float gated[];                 // [width] with gate_first
   __shared__ float scratch[33];
   const long long t = blockIdx.x;
   const float* row = y + t * width;
+  if (gate_first) {
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+      const float g = gate[t * gate_stride + i];
+      gated[i] = row[i] * ((gate_silu ? g : 1.f) / (1.f + expf(-g)));
+    }
+    __syncthreads();
+    row = gated;
+    gate = nullptr;
+  }
   auto finish = [&](int i, float r) {
     float v = row[i] * r;
     if (w) v *= widen(w[i]);
@@ -490,14 +670,16 @@ norm_gate_kernel(const float* __restrict__ y, const W* __restrict__ w,
     }
     out[t * width + i] = narrow<C>(v * scale);
   };
-  if (group == width) {
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
-    const float r = 1.f / sqrtf(block_sum(ss, scratch) / static_cast<float>(width) + eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) finish(i, r);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  if (width / group < warps) {                     // few and long parts: the whole block a part
+    for (int g0 = 0; g0 < width; g0 += group) {
+      float ss = 0.f;
+      for (int i = threadIdx.x; i < group; i += blockDim.x) ss = fmaf(row[g0 + i], row[g0 + i], ss);
+      const float r = 1.f / sqrtf(block_sum(ss, scratch) / static_cast<float>(group) + eps);
+      for (int i = threadIdx.x; i < group; i += blockDim.x) finish(g0 + i, r);
+    }
     return;
   }
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   for (int g0 = warp * group; g0 < width; g0 += warps * group) {
     float ss = 0.f;
     for (int i = lane; i < group; i += 32) ss = fmaf(row[g0 + i], row[g0 + i], ss);
@@ -720,20 +902,85 @@ SAKV_EXPORT int sakv_decay_attention(const float* proj, long long stride, int q_
 #undef SAKV_FADE
 }
 
+// xbc: [tokens, stride] of `c_dtype` with x at column x_off (heads * vdim), B at b_off and C at
+// c_off (groups * dim each); dt: fp32 rows `dt_stride` apart (a column a head); dt_bias, a (the
+// negative decay rates), d_skip: fp32 [heads]; state: fp32 [slots, heads, vdim, dim]. out: fp32
+// [tokens, heads * vdim]. Runs (chunk_len > 0) as in `sakv_selective_scan`, with dt_sums
+// [sequences, max_chunks, heads].
+SAKV_EXPORT int sakv_dual_scan(const void* xbc, int c_dtype, long long stride, int x_off, int b_off,
+                               int c_off, const float* dt, long long dt_stride,
+                               const float* dt_bias, const float* a, const float* d_skip,
+                               float* state, const int32_t* cu_seqlens, const int32_t* slots,
+                               float* out, int tokens, int sequences, int heads, int groups,
+                               int dim, int vdim, int keep_state, int chunk_len, int max_chunks,
+                               float* scratch, float* dt_sums, cudaStream_t stream) {
+  if (tokens < 0 || sequences < 0 || heads <= 0 || groups <= 0 || heads % groups || dim <= 0 ||
+      dim > 256 || vdim <= 0)
+    return cudaErrorInvalidValue;
+  if (tokens == 0 || sequences == 0) return 0;
+  const bool runs = chunk_len > 0;
+  if (runs && (max_chunks <= 0 || scratch == nullptr || dt_sums == nullptr ||
+               (long long)sequences * max_chunks > 65535))
+    return cudaErrorInvalidValue;
+  const long long walks = runs ? (long long)sequences * max_chunks : sequences;
+  const int rp = dim < 128 ? 4 : 8;        // (rows a lane; 16 lanes a column from 128 rows on)
+  const int rs = lanes_for(dim, rp);
+  int cols = 256 / rs;                       // value columns a block
+  while (cols > 1 && (long long)((vdim + cols - 1) / cols) * heads * walks < 2LL * sm_count())
+    cols /= 2;
+  while (cols > 1 && cols / 2 >= vdim) cols /= 2;
+  if (cols * rs < 32) cols = 32 / rs;        // whole warps
+  const dim3 grid((unsigned)((vdim + cols - 1) / cols), (unsigned)heads, (unsigned)walks);
+  const size_t smem = (size_t)kRun * (2 * rs * rp + cols + 2) * sizeof(float);
+#define SAKV_DUAL(RP, PHASE, C)                                                                  \
+  launch_ordered(dual_scan_kernel<RP, PHASE, C>, grid, dim3(cols * rs), smem, stream,            \
+                 DualScan<C>{(const C*)xbc, stride, x_off, b_off, c_off, dt, dt_stride, dt_bias, \
+                             a, d_skip, state, cu_seqlens, slots, out, heads, groups, dim, vdim, \
+                             rs, cols, keep_state, chunk_len, max_chunks, scratch, dt_sums})
+#define SAKV_DUAL_ALL(RP, C)                                                                     \
+  do {                                                                                           \
+    if (!runs) return SAKV_DUAL(RP, 0, C);                                                       \
+    int code = SAKV_DUAL(RP, 1, C);                                                              \
+    if (code) return code;                                                                       \
+    const long long per_head = (long long)vdim * dim;                                            \
+    const long long count = (long long)sequences * heads * per_head;                             \
+    code = launch_ordered(dual_carry_kernel, dim3((unsigned)((count + 127) / 128)), dim3(128),   \
+                          0, stream, a, state, scratch, (const float*)dt_sums, cu_seqlens,       \
+                          slots, sequences, heads, per_head, chunk_len, max_chunks, keep_state); \
+    if (code) return code;                                                                       \
+    return SAKV_DUAL(RP, 2, C);                                                                  \
+  } while (0)
+  if (c_dtype == SAKV_F32) {
+    if (rp == 4) SAKV_DUAL_ALL(4, float);
+    SAKV_DUAL_ALL(8, float);
+  }
+  if (c_dtype == SAKV_BF16) {
+    if (rp == 4) SAKV_DUAL_ALL(4, __nv_bfloat16);
+    SAKV_DUAL_ALL(8, __nv_bfloat16);
+  }
+#undef SAKV_DUAL_ALL
+#undef SAKV_DUAL
+  return cudaErrorInvalidValue;
+}
+
 // y: fp32 [tokens, width]; w: [width] of `w_dtype` (null: no weight); gate: fp32 rows
 // `gate_stride` apart (null: none), used as sigmoid(g), or g sigmoid(g) with `gate_silu`.
 // group: how many numbers share a root mean square (width: the whole row; it divides width).
+// gate_first: the gate multiplies y before the root mean square is taken, not after.
 // out: [tokens, width] of `out_dtype`.
 SAKV_EXPORT int sakv_norm_gate(const float* y, const void* w, int w_dtype, const float* gate,
                                long long gate_stride, void* out, int out_dtype, int tokens,
-                               int width, int group, int gate_silu, float eps, float scale,
-                               cudaStream_t stream) {
-  if (tokens < 0 || width <= 0 || group <= 0 || width % group) return cudaErrorInvalidValue;
+                               int width, int group, int gate_silu, int gate_first, float eps,
+                               float scale, cudaStream_t stream) {
+  if (tokens < 0 || width <= 0 || group <= 0 || width % group ||
+      (gate_first && (gate == nullptr || width > 12000)))
+    return cudaErrorInvalidValue;
   if (tokens == 0) return 0;
 #define SAKV_NG(W, C)                                                                            \
-  return launch_ordered(norm_gate_kernel<W, C>, dim3(tokens), dim3(256), 0, stream, y,           \
-                        (const W*)w, gate, gate_stride, (C*)out, width, group, gate_silu, eps,     \
-                        scale)
+  return launch_ordered(norm_gate_kernel<W, C>, dim3(tokens), dim3(256),                         \
+                        gate_first ? (size_t)width * sizeof(float) : 0, stream, y,               \
+                        (const W*)w, gate, gate_stride, (C*)out, width, group, gate_silu,        \
+                        gate_first, eps, scale)
   if (w_dtype == SAKV_F32 && out_dtype == SAKV_F32) SAKV_NG(float, float);
   if (w_dtype == SAKV_BF16 && out_dtype == SAKV_BF16) SAKV_NG(__nv_bfloat16, __nv_bfloat16);
   if (w_dtype == SAKV_BF16 && out_dtype == SAKV_F32) SAKV_NG(__nv_bfloat16, float);

@@ -39,6 +39,8 @@ class DecoderModel:
     def tensor_decls(self) -> list[TensorDecl]:
         spec = self.spec
         decls = [TensorDecl(spec.embed_name, (spec.vocab_size, spec.hidden))]
+        if spec.position_name:
+            decls.append(TensorDecl(spec.position_name, (spec.max_positions, spec.hidden)))
         for block in self.blocks:
             decls += block.tensor_decls()
         decls += self.final_norm.tensor_decls()
@@ -67,6 +69,7 @@ class DecoderModel:
         self.embed = arena.view(self.spec.embed_name)
         self.head = self.embed if self.spec.tie_head else arena.view(self.spec.head_name)
         self.head_bias = arena.view(self.spec.head_bias_name) if self.spec.head_bias_name else None
+        self.positions = arena.view(self.spec.position_name) if self.spec.position_name else None
         self.input_mix = arena.view(self.spec.input_mix_name) if self.spec.input_mix_name else None
         for block in self.blocks:
             block.bind(arena)
@@ -110,14 +113,10 @@ class DecoderModel:
         if streams > 1:          # every stream starts as the embedding's output
             x = torch.empty((streams, step.tokens, self.spec.hidden), dtype=torch.float32,
                             device=self.device)
-            ops.embed(step.token_ids, self.embed, out=x[0])
-            if self.spec.embed_scale != 1.0:
-                ops.scale_cap_(x[0], self.spec.embed_scale)
+            self._embed(step, x[0])
             ops.streams_spread(x)
         else:
-            x = ops.embed(step.token_ids, self.embed)
-            if self.spec.embed_scale != 1.0:
-                ops.scale_cap_(x, self.spec.embed_scale)
+            x = self._embed(step)
 
         def stream(x):           # what the streams stand for: their sum
             return ops.streams_step(x, reduce=True) if x.dim() == 3 else x.clone()
@@ -159,6 +158,15 @@ class DecoderModel:
         if pending is not None:
             _settle(x, pending)
         return ops.streams_step(x, reduce=True) if x.dim() == 3 else x
+
+    def _embed(self, step, out=None) -> torch.Tensor:
+        """The stream at the start: the tokens' rows of the embedding times its scale, plus
+        the learned vectors of their positions where the model has them."""
+        if self.positions is not None and step.max_position >= self.positions.shape[0]:
+            raise ValueError(f"position {step.max_position} is beyond the model's "
+                             f"{self.positions.shape[0]} learned positions")
+        return ops.embed(step.token_ids, self.embed, out=out, scale=self.spec.embed_scale,
+                         positions=step.positions, position_table=self.positions)
 
     def final_states(self, x: torch.Tensor) -> torch.Tensor:
         """The stream after the final norm, fp32 [T, hidden]: the last entry of the captured

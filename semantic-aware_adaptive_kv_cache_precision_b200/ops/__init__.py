@@ -16,7 +16,7 @@ from .linear import Deferred, gated_up, linear, per_head
 from . import gemm_tc
 from .streams import streams_spread, streams_step, token_shift
 from .recurrent import delta_rule
-from .scan import causal_conv, decay_attention, norm_gate, selective_scan, step_size
+from .scan import causal_conv, decay_attention, dual_scan, norm_gate, selective_scan, step_size
 from . import mixture
 from .mixture import latent_prepare, rotate_heads
 from .attention import (attention_decode, attention_prefill, attention_prefill_tc, decode_splits,
@@ -30,8 +30,8 @@ __all__ = ["CACHE_BLOCK", "KernelError", "embed", "rms_norm", "rope_store", "att
            "decode_splits", "plan_token_blocks", "fast_path_takes", "forget_descriptors",
            "kernel_errors", "gated_silu", "gelu_tanh", "streams_step", "streams_spread", "token_shift",
            "delta_rule", "kv_store", "layer_norm", "cached_attention", "mixture", "latent_prepare",
-           "rotate_heads", "distance_attention", "rms_update", "qk_prepare", "causal_conv",
-           "decay_attention", "norm_gate", "selective_scan", "step_size", "gated_up", "gemm_tc", "add_into", "scale_cap_", "linear", "per_head", "choose", "Deferred"]
+           "rotate_heads", "distance_attention", "rms_update", "rms_join", "qk_prepare", "causal_conv",
+           "decay_attention", "dual_scan", "norm_gate", "selective_scan", "step_size", "gated_up", "gemm_tc", "add_into", "scale_cap_", "linear", "per_head", "choose", "Deferred"]
 
 
 def _check(cond: bool, message: str) -> None:
@@ -39,9 +39,13 @@ def _check(cond: bool, message: str) -> None:
         raise KernelError(message)
 
 
-def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
-    """fp32 rows of `table` for int32 `ids`; an id outside the table gives zeros."""
-    require_cuda(ids, table)
+def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None = None,
+          scale: float = 1.0, positions: torch.Tensor | None = None,
+          position_table: torch.Tensor | None = None) -> torch.Tensor:
+    """fp32 rows of `table` for int32 `ids`, times `scale`; an id outside the table gives
+    zeros. With `position_table` ([rows, hidden] of the table's type) and `positions` (int32
+    [T]): plus the position's row, as it is."""
+    require_cuda(ids, table, positions, position_table)
     _check(ids.dtype == torch.int32 and ids.dim() == 1 and ids.is_contiguous(), "ids: int32 [T]")
     _check(table.dim() == 2 and table.is_contiguous(), "table: contiguous [vocab, hidden]")
     vocab, hidden = table.shape
@@ -49,8 +53,17 @@ def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None = Non
         out = torch.empty((ids.numel(), hidden), dtype=torch.float32, device=ids.device)
     _check(out.dtype == torch.float32 and out.is_contiguous() and out.shape == (ids.numel(), hidden),
            "out: fp32 [T, hidden]")
+    if position_table is not None:
+        _check(position_table.dtype == table.dtype and position_table.dim() == 2
+               and position_table.is_contiguous() and position_table.shape[1] == hidden,
+               "position_table: contiguous [rows, hidden] of the table's type")
+        _check(positions is not None and positions.dtype == torch.int32
+               and positions.is_contiguous() and positions.numel() == ids.numel(),
+               "positions: int32 [T]")
     call("sakv_embed", ptr(ids), ptr(table), dtype_code(table.dtype), ptr(out), ids.numel(),
-         hidden, vocab)
+         hidden, vocab, float(scale), ptr(position_table),
+         ptr(positions) if position_table is not None else None,
+         0 if position_table is None else position_table.shape[0])
     return out
 
 
@@ -282,20 +295,54 @@ def rms_update(x: torch.Tensor, y: torch.Tensor | None = None,
     return out
 
 
+def rms_join(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
+             alpha: float = 1.0, scale: float = 1.0, branch_weight: torch.Tensor | None = None,
+             other: torch.Tensor | None = None, other_weight: torch.Tensor | None = None,
+             branch_eps: float = 0.0, out_dtype: torch.dtype | None = None) -> torch.Tensor | None:
+    """In one pass over rows of the fp32 stream `x` (in place): `x <- v / rms(v) * weight` with `v
+    = alpha x + scale (n(y) + n(other))`, where n(y) is `y / rms(y) * branch_weight` (root mean
+    square with `branch_eps`), or y itself without branch weights; `other` may be absent. With
+    `out_dtype` (not fp32), returns the new stream in that type as well."""
+    require_cuda(x, y, weight, branch_weight, other, other_weight)
+    _check(x.dtype == torch.float32 and x.dim() == 2 and x.is_contiguous(), "x: fp32 [T, hidden]")
+    hidden = x.shape[1]
+    for t in (y, other):
+        _check(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == x.shape),
+               "y, other: fp32 like x")
+    for w in (weight, branch_weight, other_weight):
+        _check(w is None or (w.shape == (hidden,) and w.is_contiguous() and w.dtype == weight.dtype),
+               "weights: [hidden] of one type")
+    _check(other_weight is None or other is not None, "other_weight goes with other")
+    _check(other is None or (branch_weight is None) == (other_weight is None),
+           "both branches are normed, or neither")
+    out = None if out_dtype is None else torch.empty_like(x, dtype=out_dtype)
+    call("sakv_rms_join", ptr(x), ptr(y), ptr(branch_weight), ptr(other), ptr(other_weight),
+         float(branch_eps), float(scale), float(alpha), ptr(weight), dtype_code(weight.dtype),
+         float(eps), ptr(out), dtype_code(out_dtype if out_dtype is not None else torch.float32),
+         x.shape[0], hidden)
+    return out
+
+
 def qk_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_heads: int,
                dim: int, vdim: int, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None,
                eps: float, cos: torch.Tensor | None, sin: torch.Tensor | None,
                positions: torch.Tensor, token_seq: torch.Tensor, block_table: torch.Tensor,
                k_cache: torch.Tensor, v_cache: torch.Tensor, out_dtype: torch.dtype,
-               write_cache: bool = True) -> torch.Tensor:
+               write_cache: bool = True, norm: str | None = "whole",
+               temperature: torch.Tensor | None = None) -> torch.Tensor:
     """From a fused projection's fp32 output `proj` [T, columns] (queries at `q_off`, keys at
     `k_off`, values at `v_off`): queries and keys each divided by the root mean square of their
     whole projection and multiplied by `q_weight` / `k_weight` (None: no norm), the first
     `2 * cos.shape[1]` numbers of every head turned by the token's position (None: no
     rotation), keys and values stored in the cache blocks. Returns the queries [T, heads *
-    dim] of `out_dtype`."""
+    dim] of `out_dtype`. `norm` "head": every head is divided by its own root mean square
+    (`q_weight`, `k_weight`: [dim], the same for all heads, or None: no weight).
+    `temperature` (fp32 [positions]): queries are multiplied by their position's number."""
     require_cuda(proj, q_weight, k_weight, cos, sin, positions, token_seq, block_table, k_cache,
-                 v_cache)
+                 v_cache, temperature)
+    _check(norm in (None, "whole", "head"), "norm: 'whole', 'head' or None")
+    _check(temperature is None or (temperature.dtype == torch.float32 and temperature.dim() == 1
+                                   and temperature.is_contiguous()), "temperature: fp32 [positions]")
     tokens = proj.shape[0]
     _check(proj.dtype == torch.float32 and proj.dim() == 2 and proj.stride(1) == 1,
            "proj: fp32 [T, columns] with contiguous rows")
@@ -303,9 +350,10 @@ def qk_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: in
            <= proj.shape[1], "queries, keys or values reach beyond proj's columns")
     _check((q_weight is None) == (k_weight is None), "q_weight and k_weight come together")
     if q_weight is not None:
-        _check(q_weight.shape == (heads * dim,) and k_weight.shape == (kv_heads * dim,)
+        _check(((q_weight.shape == (heads * dim,) and k_weight.shape == (kv_heads * dim,))
+                if norm == "whole" else q_weight.shape == k_weight.shape == (dim,))
                and q_weight.is_contiguous() and k_weight.is_contiguous()
-               and q_weight.dtype == k_weight.dtype, "norm weights: [heads * dim], [kv_heads * dim]")
+               and q_weight.dtype == k_weight.dtype, "norm weights: [heads * dim], [kv_heads * dim] (a norm a head: [dim])")
     rot = 0
     if cos is not None:
         _check(cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.dim() == 2
@@ -326,7 +374,8 @@ def qk_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: in
          ptr(q_weight), ptr(k_weight), dtype_code(q_weight.dtype) if q_weight is not None else F32,
          float(eps), ptr(cos), ptr(sin), rot, ptr(positions), ptr(token_seq), ptr(block_table),
          block_table.shape[1], ptr(q), ptr(k_cache), ptr(v_cache), dtype_code(out_dtype), tokens,
-         heads, kv_heads, dim, vdim, int(write_cache))
+         heads, kv_heads, dim, vdim, int(write_cache),
+         2 if norm == "head" else 1 if norm and q_weight is not None else 0, ptr(temperature))
     return q
 
 
@@ -339,7 +388,8 @@ def cached_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      splits: int = 1, key_splits: int = 1, warp_stage: bool = False,
                      heads_first: bool = False, keep_first: int = 0,
                      sink: torch.Tensor | None = None,
-                     head_gate: torch.Tensor | None = None) -> torch.Tensor:
+                     head_gate: torch.Tensor | None = None,
+                     elem_gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of every token of the step over its sequence's cache, in the general
     form of `csrc/attention_distance.cu`: scores, softmax weights and weighted sums in fp32.
 
@@ -353,7 +403,8 @@ def cached_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     with a window, `keep_first` k: the keys at positions below k stay visible to every later
     query. `sink` (fp32 [heads]): the softmax's denominator of head h also holds
     `exp(sink[h])`. With one map the output is multiplied by `out_scale`, and with `head_gate`
-    ([T, heads] of q's type, any row stride) head h's by `sigmoid(head_gate[t, h])`. Two
+    ([T, heads] of q's type, any row stride) head h's by `sigmoid(head_gate[t, h])`, with
+    `elem_gate` (fp32 [T, heads * vdim], any row stride) element by element by its sigmoid. Two
     maps are combined as `a1 - lam * a2`, divided by their root mean square over vdim (+ eps),
     times `out_scale`, times the sigmoid of the `vdim` numbers that lie `gate_elem_off + h *
     vdim` elements after the token's first query. Returns [T, heads * vdim] of q's type.
@@ -365,8 +416,13 @@ def cached_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     are ONE token's groups of heads and share every chunk of its keys through shared memory, so
     the rows are read once for all the token's heads; `key_splits` blocks a token then take
     contiguous shares of the chunks."""
-    require_cuda(q, k_cache, v_cache, positions, token_seq, block_table, q2, sink, head_gate)
+    require_cuda(q, k_cache, v_cache, positions, token_seq, block_table, q2, sink, head_gate,
+                 elem_gate)
     tokens = q.shape[0]
+    _check(elem_gate is None or (maps == 1 and elem_gate.dtype == torch.float32
+                                 and elem_gate.shape == (tokens, heads * vdim)
+                                 and elem_gate.stride(1) == 1),
+           "elem_gate: fp32 [T, heads * vdim] with contiguous rows, one map")
     _check(head_gate is None or (maps == 1 and head_gate.dtype == q.dtype and head_gate.dim() == 2
                                  and head_gate.shape == (tokens, heads)
                                  and head_gate.stride(1) == 1),
@@ -417,7 +473,8 @@ def cached_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
          float(out_scale), float(eps), -1 if gate_elem_off is None else int(gate_elem_off),
          int(splits), int(key_splits), ptr(scratch), floats, ptr(tickets), int(warp_stage),
          int(heads_first), int(keep_first) if window else 0, ptr(sink), ptr(head_gate),
-         0 if head_gate is None else head_gate.stride(0))
+         0 if head_gate is None else head_gate.stride(0), ptr(elem_gate),
+         0 if elem_gate is None else elem_gate.stride(0))
     return out
 
 

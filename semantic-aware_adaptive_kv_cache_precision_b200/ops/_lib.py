@@ -21,7 +21,7 @@ P, I, L, F, U = c_void_p, c_int, c_longlong, c_float, c_ulonglong
 
 #: exported function -> (library, argument types); the stream is always last
 SIGNATURES = {
-    "sakv_embed": ("elementwise", [P, P, I, P, I, I, I, P]),
+    "sakv_embed": ("elementwise", [P, P, I, P, I, I, I, F, P, P, I, P]),
     "sakv_gated_silu": ("elementwise", [P, P, I, I, I, P]),
     "sakv_add_into": ("elementwise", [P, P, I, L, P]),
     "sakv_scale_cap": ("elementwise", [P, L, F, F, P]),
@@ -37,10 +37,11 @@ SIGNATURES = {
                                 [P, I, L, I, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P]),
     "sakv_cached_attention": ("attention_distance",
                               [P, I, L, I, P, L, I, I, I, P, P, I, P, I, P, P, P, I, I, I, I, I, I,
-                               I, F, I, I, F, F, F, I, I, I, P, L, P, I, I, I, P, P, L, P]),
+                               I, F, I, I, F, F, F, I, I, I, P, L, P, I, I, I, P, P, L, P, L, P]),
     "sakv_rms_update": ("norm_update", [P, P, P, F, P, P, F, I, P, I, I, I, F, P]),
+    "sakv_rms_join": ("norm_update", [P, P, P, P, P, F, F, F, P, I, F, P, I, I, I, P]),
     "sakv_qk_prepare": ("qk_prepare", [P, L, I, I, I, P, P, I, F, P, P, I, P, P, P, I, P, P, P,
-                                       I, I, I, I, I, I, I, P]),
+                                       I, I, I, I, I, I, I, I, P, P]),
     "sakv_causal_conv": ("recurrent_scan", [P, L, P, P, I, P, P, P, P, P, I, I, I, I, P]),
     "sakv_conv_state": ("recurrent_scan", [P, L, P, P, P, I, I, I, P]),
     "sakv_step_size": ("recurrent_scan", [P, L, I, P, P, I, P, I, I, P]),
@@ -49,18 +50,20 @@ SIGNATURES = {
     "sakv_conv_step": ("recurrent_scan", [P, L, P, P, I, P, P, P, I, I, I, I, I, P]),
     "sakv_decay_attention": ("recurrent_scan", [P, L, I, I, I, P, P, P, P, P, I, I, I, I, I, I,
                                                 I, I, P, I, I, P, P, P, F, P]),
-    "sakv_norm_gate": ("recurrent_scan", [P, P, I, P, L, P, I, I, I, I, I, F, F, P]),
+    "sakv_dual_scan": ("recurrent_scan", [P, I, L, I, I, I, P, L, P, P, P, P, P, P, P, I, I, I, I, I,
+                                          I, I, I, I, P, P, P]),
+    "sakv_norm_gate": ("recurrent_scan", [P, P, I, P, L, P, I, I, I, I, I, I, F, F, P]),
     "sakv_layer_norm": ("layer_norm", [P, P, P, P, P, I, P, I, I, I, F, P]),
     "sakv_latent_prepare": ("latent", [P, L, I, I, I, P, P, I, F, P, P, P, I, P, P, P, P, I, I, I,
                                        I, P]),
     "sakv_rotate_heads": ("latent", [P, I, L, I, I, I, I, P, P, P, I, I, P]),
     "sakv_moe_logits": ("moe", [P, I, P, P, I, I, I, P]),
-    "sakv_moe_route": ("moe", [P, L, I, I, P, P, P, P, I, I, I, P, P]),
+    "sakv_moe_route": ("moe", [P, L, I, I, P, P, P, P, I, I, I, P, I, I, I, P]),
     "sakv_moe_plan": ("moe", [P, P, P, P, P, I, I, P]),
-    "sakv_moe_route_plan": ("moe", [P, L, I, I, P, P, P, I, I, I, P, P, P, P, P, I, P]),
+    "sakv_moe_route_plan": ("moe", [P, L, I, I, P, P, P, I, I, I, P, I, I, I, P, P, P, P, I, P]),
     "sakv_moe_gather": ("moe", [P, I, P, P, P, P, P, P, I, I, I, I, P]),
-    "sakv_moe_product": ("moe", [P, I, P, P, L, P, P, P, P, I, P, I, I, I, F, F, P]),
-    "sakv_clamped_act": ("moe", [P, P, I, I, I, F, F, P]),
+    "sakv_moe_product": ("moe", [P, I, P, P, L, P, P, P, P, I, P, I, I, I, F, F, F, P]),
+    "sakv_clamped_act": ("moe", [P, P, I, I, I, F, F, F, P]),
     "sakv_moe_combine": ("moe", [P, P, P, I, P, P, L, P, I, I, I, P, I, I, P]),
     "sakv_rmsnorm": ("norm", [P, P, I, L, P, P, I, P, I, I, I, F, P]),
     "sakv_rope_store": ("rope", [P, I, L, P, P, P, I, P, P, I, P, P, I, I, I, I, I, P]),
@@ -74,9 +77,9 @@ SIGNATURES = {
                                [P, P, P, L, P, P, I, P, P, I, I, I, I, F, I, P]),
     "sakv_prefill_attention_tc": ("attention_prefill_tc",
                                   [P, P, P, P, P, I, P, I, P, P, P, P, I, I, I, I, F, I, P]),
-    "sakv_gemm_tc": ("gemm_tc", [P, P, I, I, I, I, I, I, I, I, P, I, P, L, L, P]),
+    "sakv_gemm_tc": ("gemm_tc", [P, P, I, I, I, I, I, I, I, I, P, I, P, L, L, F, F, F, P]),
     "sakv_gemm_wide": ("gemm_wide", [P, P, I, I, I, I, P, L, P]),
-    "sakv_gemm_pair": ("gemm_pair", [P, P, I, I, I, I, P, L, P]),
+    "sakv_gemm_pair": ("gemm_pair", [P, P, I, I, I, I, P, L, I, F, F, F, P]),
     "sakv_lib_accumulate": ("gemm_lib", [P, L, P, P, L, I, I, I, P, L, P]),
 }
 

@@ -9,7 +9,7 @@ import torch
 
 from ._lib import BF16, F32, KernelError, call, dtype_code, plain_function, ptr, sm_count
 
-EPI_BF16, EPI_F32, EPI_ACCUM, EPI_GATED = 0, 1, 2, 3
+EPI_BF16, EPI_F32, EPI_ACCUM, EPI_GATED, EPI_CLAMPED = 0, 1, 2, 3, 4
 
 _weight_maps: dict = {}
 MAX_PARTS = 16      # K ranges whose sums the reader adds
@@ -101,13 +101,15 @@ def choose_parts(m: int, n: int, k: int) -> tuple:
 
 
 def gemm(x: torch.Tensor, weight: torch.Tensor, bias, epi: int, out: torch.Tensor,
-         n: int, dual_offset: int = 0, splits: int | None = None, parts: int = 1) -> torch.Tensor:
+         n: int, dual_offset: int = 0, splits: int | None = None, parts: int = 1,
+         clamp: tuple = (0.0, 0.0, 0.0)) -> torch.Tensor:
     """`out` is written (EPI_BF16, EPI_F32, EPI_GATED) or added to (EPI_ACCUM); `n` is the
     number of output columns (rows of `weight`, or half of them for EPI_GATED). With
     `parts` > 1 (EPI_F32, `out` [parts, M, n]) K is cut into that many ranges whose sums are
-    left apart in `out[i]`, with the bias in `out[0]`."""
+    left apart in `out[i]`, with the bias in `out[0]`. `clamp`: EPI_CLAMPED's (limit, alpha,
+    plus)."""
     m, k = x.shape
-    dual = epi == EPI_GATED
+    dual = epi in (EPI_GATED, EPI_CLAMPED)
     mt = token_tile(m, dual)
     n_tiles, m_tiles = -(-n // 128), -(-m // mt)
     if parts > 1:
@@ -119,7 +121,7 @@ def gemm(x: torch.Tensor, weight: torch.Tensor, bias, epi: int, out: torch.Tenso
     x_raw, x_map = _make_map(x, mt)
     call("sakv_gemm_tc", _weight_map(weight), x_map, m, n, k, mt, splits, parts, epi, dual_offset,
          ptr(bias), dtype_code(bias.dtype) if bias is not None else BF16, ptr(out),
-         out.stride(-2), out.stride(0) if parts > 1 else 0)
+         out.stride(-2), out.stride(0) if parts > 1 else 0, *(float(c) for c in clamp))
     return out
 
 

@@ -101,15 +101,18 @@ def gated(x: torch.Tensor, w_gate_up: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def gated_pair(x: torch.Tensor, w_gate_up: torch.Tensor) -> torch.Tensor:
-    """The same product on pairs of SMs (`csrc/gemm_pair.cu`, tcgen05 with `cta_group::2`)."""
+def gated_pair(x: torch.Tensor, w_gate_up: torch.Tensor,
+               clamp: tuple | None = None) -> torch.Tensor:
+    """The same product on pairs of SMs (`csrc/gemm_pair.cu`, tcgen05 with `cta_group::2`); with
+    `clamp` (limit, alpha, plus) the clamped activation instead of the gated silu."""
     inter = w_gate_up.shape[0] // 2
     if inter % 8:
         raise KernelError("gemm_wide.gated_pair: the intermediate size must be a multiple of 8")
     out = torch.empty((x.shape[0], inter), dtype=torch.bfloat16, device=x.device)
     x_raw, x_map = _make_map(x, "sakv_gemm_pair_map")
     call("sakv_gemm_pair", x_map, _weight_map(w_gate_up, "sakv_gemm_pair_map"), x.shape[0], inter, x.shape[1], inter,
-         ptr(out), out.stride(0))
+         ptr(out), out.stride(0), int(clamp is not None),
+         *(float(c) for c in (clamp or (0.0, 0.0, 0.0))))
     return out
 
 

@@ -68,21 +68,27 @@ class Deferred:
         self.delta = delta
 
 
-def gated_up(x: torch.Tensor, w_gate_up: torch.Tensor) -> torch.Tensor:
+def gated_up(x: torch.Tensor, w_gate_up: torch.Tensor, clamp: tuple | None = None) -> torch.Tensor:
     """`silu(x Wgate^T) * (x Wup^T)` for `w_gate_up = [Wgate; Wup]`: one kernel with the
     activation in its epilogue where the tensor-core kernel takes the operands, else the
-    product followed by the activation kernel."""
+    product followed by the activation kernel. With `clamp` (limit, alpha, plus): `g *
+    sigmoid(alpha g) * (u + plus)` instead, g = min(gate, limit), u = up within +-limit."""
     from . import gated_silu
+    from .mixture import clamped_act
     inter = w_gate_up.shape[0] // 2
     if x.shape[0] <= TC_MAX_TOKENS and inter % 128 == 0 and gemm_tc.takes(x, w_gate_up):
         out = torch.empty((x.shape[0], inter), dtype=torch.bfloat16, device=x.device)
+        if clamp is not None:
+            return gemm_tc.gemm(x, w_gate_up, None, gemm_tc.EPI_CLAMPED, out, inter,
+                                dual_offset=inter, clamp=clamp)
         return gemm_tc.gemm(x, w_gate_up, None, gemm_tc.EPI_GATED, out, inter, dual_offset=inter)
     if inter % 8 == 0 and gemm_wide.takes(x, w_gate_up):
         if gemm_wide.pair_worth_it(x.shape[0]) and gemm_wide.resident_pairs() > 0:
-            return gemm_wide.gated_pair(x, w_gate_up)
-        if gemm_wide.worth_it(x.shape[0], inter):
+            return gemm_wide.gated_pair(x, w_gate_up, clamp)
+        if clamp is None and gemm_wide.worth_it(x.shape[0], inter):
             return gemm_wide.gated(x, w_gate_up)
-    return gated_silu(linear(x, w_gate_up, out_dtype=x.dtype))
+    both = linear(x, w_gate_up, out_dtype=x.dtype)
+    return gated_silu(both) if clamp is None else clamped_act(both, *clamp)
 
 
 def per_head(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> torch.Tensor:

@@ -46,12 +46,16 @@ def router_logits(h: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 
 
 def route(logits: torch.Tensor, experts: int, top: int, identity: int = 0,
-          softmax: bool = False, bias: torch.Tensor | None = None) -> Routing:
+          softmax: bool = False, bias: torch.Tensor | None = None, groups: int = 1,
+          keep_groups: int = 1, renormalize: bool = False) -> Routing:
     """logits: fp32 [T, >= experts + identity]; the `top` largest scores among the first
     `experts + identity` columns a row. The score is the sigmoid of the logit, or with
     `softmax` the softmax over those columns; `bias` (fp32 [experts + identity]) is added for
     the choice only. A choice among the last `identity` columns is an identity expert: it gets
-    no row in the grouped products, and `combine` adds the token's input times its weight."""
+    no row in the grouped products, and `combine` adds the token's input times its weight.
+    `groups` g (up to 64): the columns form g equal groups of neighbours, and only those of the
+    `keep_groups` groups with the largest best score can be chosen. `renormalize`: the weights
+    are the chosen scores divided by (their sum + 1e-20)."""
     require_cuda(logits, bias)
     outputs = experts + identity
     _check(logits.dtype == torch.float32 and logits.dim() == 2 and logits.stride(1) == 1
@@ -76,10 +80,12 @@ def route(logits: torch.Tensor, experts: int, top: int, identity: int = 0,
     if 0 < tokens <= ROUTE_IN_ONE_BLOCK:
         call("sakv_moe_route_plan", ptr(logits), logits.stride(0), outputs, top, ptr(r.chosen),
              ptr(r.weights), ptr(r.rank), tokens, experts, int(bool(softmax)), ptr(bias),
+             int(groups), int(keep_groups), int(bool(renormalize)),
              ptr(r.offsets), ptr(r.tile_expert), ptr(r.tile_row), ptr(r.n_tiles), r.max_tiles)
         return r
     call("sakv_moe_route", ptr(logits), logits.stride(0), outputs, top, ptr(r.chosen),
-         ptr(r.weights), ptr(counts), ptr(r.rank), tokens, experts, int(bool(softmax)), ptr(bias))
+         ptr(r.weights), ptr(counts), ptr(r.rank), tokens, experts, int(bool(softmax)), ptr(bias),
+         int(groups), int(keep_groups), int(bool(renormalize)))
     call("sakv_moe_plan", ptr(counts), ptr(r.offsets), ptr(r.tile_expert), ptr(r.tile_row),
          ptr(r.n_tiles), experts, r.max_tiles)
     return r
@@ -98,10 +104,10 @@ def gather_rows(h: torch.Tensor, r: Routing, weight_input: bool) -> torch.Tensor
 
 
 def grouped_product(rows: torch.Tensor, r: Routing, w0: torch.Tensor, w1: torch.Tensor | None,
-                    limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
+                    limit: float = 0.0, alpha: float = 0.0, plus: float = 1.0) -> torch.Tensor:
     """rows [R, k] sorted by expert times every expert's own weights. `w0`, `w1`: [experts, n,
-    k]. With `w1`: the clamped gated activation of the two products, [R, n] of rows' type;
-    without: the product, fp32 [R, n]."""
+    k]. With `w1`: the clamped gated activation of the two products (`clamped_act`), [R, n] of
+    rows' type; without: the product, fp32 [R, n]."""
     require_cuda(rows, w0, w1)
     _check(rows.dim() == 2 and rows.is_contiguous() and w0.dim() == 3 and w0.is_contiguous()
            and w0.shape[0] == r.experts and w0.shape[2] == rows.shape[1]
@@ -113,12 +119,13 @@ def grouped_product(rows: torch.Tensor, r: Routing, w0: torch.Tensor, w1: torch.
                       device=rows.device)
     call("sakv_moe_product", ptr(rows), dtype_code(rows.dtype), ptr(w0), ptr(w1), w0.stride(0),
          ptr(r.tile_expert), ptr(r.tile_row), ptr(r.offsets), ptr(r.n_tiles), r.max_tiles,
-         ptr(out), n, k, int(w1 is not None), float(limit), float(alpha))
+         ptr(out), n, k, int(w1 is not None), float(limit), float(alpha), float(plus))
     return out
 
 
-def clamped_act(gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
-    """`g * sigmoid(alpha g) * (u + 1)` with g = min(gate, limit), u = clamp(up, +-limit) for
+def clamped_act(gate_up: torch.Tensor, limit: float, alpha: float,
+                plus: float = 1.0) -> torch.Tensor:
+    """`g * sigmoid(alpha g) * (u + plus)` with g = min(gate, limit), u = clamp(up, +-limit) for
     `gate_up[t] = [gate | up]`."""
     require_cuda(gate_up)
     _check(gate_up.dim() == 2 and gate_up.is_contiguous() and gate_up.shape[1] % 2 == 0,
@@ -126,7 +133,7 @@ def clamped_act(gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tens
     tokens, ff = gate_up.shape[0], gate_up.shape[1] // 2
     out = torch.empty((tokens, ff), dtype=gate_up.dtype, device=gate_up.device)
     call("sakv_clamped_act", ptr(gate_up), ptr(out), dtype_code(gate_up.dtype), tokens, ff,
-         float(limit), float(alpha))
+         float(limit), float(alpha), float(plus))
     return out
 
 

@@ -1,6 +1,6 @@
 """The recurrences without feedback from the state into its own update, over a step's tokens
-(`csrc/recurrent_scan.cu`): the selective scan with its convolution and step sizes, and
-attention without softmax over a fading state with its norm and gate."""
+(`csrc/recurrent_scan.cu`): the selective scan with its convolution and step sizes, attention
+without softmax over a fading state with its norm and gate, and the state-space dual form."""
 
 from __future__ import annotations
 
@@ -170,13 +170,48 @@ def decay_attention(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, head
     return out
 
 
+def dual_scan(xbc: torch.Tensor, x_off: int, b_off: int, c_off: int, dt: torch.Tensor,
+              dt_bias: torch.Tensor, a: torch.Tensor, d_skip: torch.Tensor, heads: int,
+              groups: int, n_state: int, vdim: int, state: torch.Tensor, step,
+              keep_state: bool = True, run: int = 0) -> torch.Tensor:
+    """The state-space dual form over each sequence's tokens: per head `S <- exp(dt a) S + dt B
+    x^T; y = S^T C + d_skip x` with `dt = softplus(dt + dt_bias)`. `xbc`: [T, columns] of either
+    type with x (heads * vdim columns from `x_off`), B and C (groups * n_state each from `b_off`,
+    `c_off`; head h reads group floor(h / (heads / groups))); `dt`: fp32 [T, heads] (any row
+    stride); `dt_bias`, `a` (negative), `d_skip`: fp32 [heads]. `state`: fp32 [slots, heads, vdim,
+    n_state], read and (with `keep_state`) left. `run`: as in `selective_scan`. Returns fp32 [T,
+    heads * vdim]."""
+    require_cuda(xbc, dt, dt_bias, a, d_skip, state)
+    tokens = xbc.shape[0]
+    _check(xbc.dim() == 2 and xbc.stride(1) == 1
+           and max(x_off + heads * vdim, b_off + groups * n_state, c_off + groups * n_state)
+           <= xbc.shape[1], "xbc: [T, columns] holding x, B and C")
+    _check(heads % groups == 0, "heads must be a multiple of groups")
+    _check(dt.dtype == torch.float32 and dt.shape == (tokens, heads) and dt.stride(1) == 1,
+           "dt: fp32 [T, heads] with contiguous rows")
+    for v in (dt_bias, a, d_skip):
+        _check(v.dtype == torch.float32 and v.shape == (heads,) and v.is_contiguous(),
+               "dt_bias, a, d_skip: fp32 [heads]")
+    _check(state.dtype == torch.float32 and state.is_contiguous()
+           and tuple(state.shape[1:]) == (heads, vdim, n_state),
+           "state: fp32 [slots, heads, vdim, n_state]")
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=xbc.device)
+    runs, scratch, sums = _runs(run, step, heads * vdim * n_state, heads, xbc.device)
+    call("sakv_dual_scan", ptr(xbc), dtype_code(xbc.dtype), xbc.stride(0), int(x_off), int(b_off),
+         int(c_off), ptr(dt), dt.stride(0), ptr(dt_bias), ptr(a), ptr(d_skip), ptr(state),
+         ptr(step.cu_seqlens), ptr(step.slots), ptr(out), tokens, step.sequences, heads, groups,
+         n_state, vdim, int(keep_state), int(run) if runs else 0, runs, ptr(scratch), ptr(sums))
+    return out
+
+
 def norm_gate(y: torch.Tensor, weight: torch.Tensor | None, gate: torch.Tensor | None, eps: float,
               scale: float, out_dtype: torch.dtype, group: int | None = None,
-              gate_silu: bool = False) -> torch.Tensor:
+              gate_silu: bool = False, gate_first: bool = False) -> torch.Tensor:
     """`y / sqrt(mean(y^2) + eps) * weight * sigmoid(gate) * scale` over whole rows of fp32 `y`
     [T, width], or with `group` over each run of that many numbers of a row (a head's
     outputs); `weight` None: no weight; `gate`: fp32 [T, width] (a view with any row stride)
-    or None, used as `gate * sigmoid(gate)` with `gate_silu`."""
+    or None, used as `gate * sigmoid(gate)` with `gate_silu`. `gate_first`: the gate multiplies
+    y before the root mean square is taken instead of after."""
     require_cuda(y, weight, gate)
     tokens, width = y.shape
     group = width if group is None else int(group)
@@ -186,9 +221,10 @@ def norm_gate(y: torch.Tensor, weight: torch.Tensor | None, gate: torch.Tensor |
     _check(group > 0 and width % group == 0, "group: a divisor of the width")
     _check(gate is None or (gate.dtype == torch.float32 and gate.shape == y.shape
                             and gate.stride(1) == 1), "gate: fp32 [T, width] with contiguous rows")
+    _check(not gate_first or gate is not None, "gate_first needs a gate")
     out = torch.empty((tokens, width), dtype=out_dtype, device=y.device)
     call("sakv_norm_gate", ptr(y), ptr(weight),
          dtype_code(weight.dtype if weight is not None else torch.float32), ptr(gate),
          0 if gate is None else gate.stride(0), ptr(out), dtype_code(out_dtype), tokens, width,
-         group, int(bool(gate_silu)), float(eps), float(scale))
+         group, int(bool(gate_silu)), int(bool(gate_first)), float(eps), float(scale))
     return out

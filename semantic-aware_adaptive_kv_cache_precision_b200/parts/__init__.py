@@ -19,10 +19,12 @@ from .decay_attention import DecayAttention
 from .parallel_mixer import ParallelMixer
 from .selective_scan import SelectiveScanMixer
 from .output_norm import OutputNormBlock
+from .post_norm import PostNormBlock, PostNormUpdate
+from .dual_scan import DualScanMixer
 
 __all__ = ["Part", "build_part", "register_part", "RMSNorm", "RotaryHalf", "RotaryInterleaved", "NoPosition",
            "GQAAttention", "GatedMLP", "DenseMLP", "PreNormBlock", "DeltaRuleMixer",
            "LogDistanceAttention", "StreamBlock", "StreamUpdate", "LayerNorm", "LatentAttention",
            "DifferentialAttention", "RoutedExperts", "SandwichBlock", "NormedUpdate",
            "WindowSinkAttention", "DecayAttention", "ParallelMixer", "SelectiveScanMixer",
-           "OutputNormBlock"]
+           "OutputNormBlock", "PostNormBlock", "PostNormUpdate", "DualScanMixer"]

@@ -1,7 +1,8 @@
 """Dense gated feed-forward: `residual += down( silu(gate(h)) * up(h) )`
 (`src/microinfer/model.py:392-396`, `src/core_kernels/swiglu.cu:26-38`). Gate and
 up are one product over the rows [Wgate; Wup] laid back to back in device
-memory; the activation is fp32 inside with one rounding at its store."""
+memory; the activation is fp32 inside with one rounding at its store. The activation may
+also be the clamped one (`GatedMLPSpec`)."""
 
 from __future__ import annotations
 
@@ -15,8 +16,12 @@ from .base import Part, register_part
 class GatedMLP(Part):
     def __init__(self, spec, prefix, mode):
         super().__init__(spec, prefix, mode)
-        if spec.activation != "silu":
-            raise ValueError(f"activation {spec.activation!r}: only 'silu' is built")
+        if spec.activation not in ("silu", "clamped"):
+            raise ValueError(f"activation {spec.activation!r}: 'silu' and 'clamped' are built")
+        self.clamp = (spec.limit, spec.alpha, spec.plus) if spec.activation == "clamped" else None
+        self.kernel_libraries = ("moe" if self.clamp else "elementwise",)
+        if mode == "bfloat16":
+            self.kernel_libraries += ("gemm_tc", "gemm_pair")
         if spec.bias:
             raise ValueError("a gated feed-forward with biases is not built")
 
@@ -41,12 +46,13 @@ class GatedMLP(Part):
 
     def produce(self, h, step):
         """The feed-forward's output as a tensor of its own, fp32 [T, hidden]."""
-        return ops.linear(ops.gated_up(h, self.w_gate_up), self.w_down, out_dtype=torch.float32)
+        return ops.linear(ops.gated_up(h, self.w_gate_up, self.clamp), self.w_down,
+                          out_dtype=torch.float32)
 
     can_defer = True
 
     def forward(self, h, step, residual, defer=False):
-        act = ops.gated_up(h, self.w_gate_up)
+        act = ops.gated_up(h, self.w_gate_up, self.clamp)
         out = ops.linear(act, self.w_down, accumulate_into=residual, may_defer=defer)
         return out.delta if isinstance(out, ops.Deferred) else None
 

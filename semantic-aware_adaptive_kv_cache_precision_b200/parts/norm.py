@@ -56,6 +56,16 @@ class RMSNorm(Part):
     def complete(self, x, y):
         self.update(x, y)
 
+    def join(self, x, y, alpha, out_dtype=None, other=None, norms=None, scale=1.0):
+        """`x <- norm(alpha x + scale (y + other))` in place on the fp32 stream, y and other (may
+        be None) each normed by its own of `norms` first where given; with `out_dtype`, also
+        returns the new stream in that type."""
+        na, nb = norms or (None, None)
+        return ops.rms_join(x, y, self.weight, self.spec.eps, alpha=alpha, scale=scale,
+                            branch_weight=None if na is None else na.weight, other=other,
+                            other_weight=None if nb is None else nb.weight,
+                            branch_eps=0.0 if na is None else na.spec.eps, out_dtype=out_dtype)
+
 
 class LayerNorm(RMSNorm):
     kernel_libraries = ("layer_norm", "elementwise")

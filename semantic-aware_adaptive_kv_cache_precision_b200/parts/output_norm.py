@@ -55,6 +55,9 @@ class OutputNormBlock(Part):
     def _stream(self, x, update=None):
         """The stream as the next sublayer reads it, after it has taken up `update`."""
         same = self.act_dtype == torch.float32          # the sublayer reads the stream itself
+        if hasattr(update, "take_up"):
+            h = update.take_up(x, None if same else self.act_dtype)
+            return x if same else h
         if isinstance(update, NormedUpdate) and getattr(update.norm, "folds_update", False):
             h = update.norm.update(x, update.y, out_dtype=None if same else self.act_dtype)
             return x if same else h
@@ -65,12 +68,16 @@ class OutputNormBlock(Part):
                 ops.add_into(x, update)
         return x if same else ops.rms_update(x, out_dtype=self.act_dtype)
 
+    def _update(self, part, norm, h, step, *cache):
+        """What the sublayer `part` does to the stream, still to be taken up by it."""
+        return NormedUpdate(_run(part, h, step, *cache), norm)
+
     def forward(self, x, step, view, write_cache=True, pending=None, leave_pending=True):
         h = self._stream(x, pending)
-        update = NormedUpdate(_run(self.mixer, h, step, view, write_cache), self.mixer_after)
+        update = self._update(self.mixer, self.mixer_after, h, step, view, write_cache)
         if self.ffn is not None:
             h = self._stream(x, update)
-            update = NormedUpdate(_run(self.ffn, h, step), self.ffn_after)
+            update = self._update(self.ffn, self.ffn_after, h, step)
         if leave_pending:
             return update
         update.apply(x)

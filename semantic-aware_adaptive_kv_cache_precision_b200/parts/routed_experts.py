@@ -5,9 +5,11 @@
     token's experts; the last `identity` outputs stand for experts that return their input
     expert_e(x) = Wdown_e [ g * sigmoid(alpha g) * (u + 1) ],  g = min(Wgate_e x, limit),
                                                               u = clamp(Wup_e x, -limit, limit)
+        (or the plain gated form: limit infinite, alpha 1, and 0 in the place of the 1)
     out = sum_chosen expert_e(s_e h)  +  sigmoid(h Wsg^T) * shared(h)
 
-The chosen scores are used as they are (or divided by their sum with `renormalize`) and
+The outputs may form groups of which only the best few are open to a token. The chosen scores
+are used as they are (or divided by their sum with `renormalize`) and
 multiply the expert's INPUT (`weight_input`) or its output. Everything stays on the device:
 the router's product runs in fp32 on the step's tokens, a kernel chooses and counts, the
 tokens' rows are sorted by expert, and two grouped products (gate and up with the activation
@@ -33,9 +35,12 @@ class RoutedExperts(Part):
         super().__init__(spec, prefix, mode)
         if spec.score not in ("sigmoid", "softmax"):
             raise ValueError(f"router score {spec.score!r}: 'sigmoid' and 'softmax' are built")
-        if spec.renormalize:
-            raise ValueError("renormalized router weights are not built")
         self.outputs = spec.experts + spec.identity
+        if not 1 <= spec.groups <= 64 or self.outputs % spec.groups \
+                or not 1 <= spec.keep_groups <= spec.groups \
+                or self.outputs // spec.groups * spec.keep_groups < spec.top:
+            raise ValueError(f"{spec.groups} groups of which {spec.keep_groups} stay open do not "
+                             f"fit {self.outputs} outputs and top {spec.top}")
         if spec.experts < 1 or spec.identity < 0 or spec.top > self.outputs \
                 or self.outputs > 1024 or spec.top > 32:
             raise ValueError("the router takes up to 1024 outputs (experts and identity "
@@ -95,17 +100,18 @@ class RoutedExperts(Part):
         s = self.spec
         logits = mixture.router_logits(h, self.w_route)
         routing = mixture.route(logits, s.experts, s.top, s.identity, s.score == "softmax",
-                                self.correction)
+                                self.correction, s.groups, s.keep_groups, s.renormalize)
         # (a checkpoint stored in 32 bits keeps its matrices so: the experts then run in 32 bits)
         rows = mixture.gather_rows(h if h.dtype == self.w_gate.dtype else h.to(self.w_gate.dtype),
                                    routing, s.weight_input)
         act = mixture.grouped_product(rows, routing, self.w_gate, self.w_up, s.expert.limit,
-                                      s.expert.alpha)
+                                      s.expert.alpha, s.expert.plus)
         products = mixture.grouped_product(act, routing, self.w_down, None)
         shared = gate = None
         if s.shared is not None:
             both = ops.linear(h, self.w_shared_in, out_dtype=self.act_dtype)
-            shared = ops.linear(mixture.clamped_act(both, s.shared.limit, s.shared.alpha),
+            shared = ops.linear(mixture.clamped_act(both, s.shared.limit, s.shared.alpha,
+                                                    s.shared.plus),
                                 self.w_shared_down, out_dtype=torch.float32)
             gate = logits[:, self.outputs] if self.has_gate else None
         return mixture.combine(products, routing, not s.weight_input, shared, gate, h, into)

@@ -3,10 +3,12 @@ logit a head in the softmax's denominator (`WindowSinkAttentionSpec`):
 
     [q | k | v] = h Wfused^T + b
     q <- q / rms(q) * wq,  k <- k / rms(k) * wk      (over the WHOLE projection, all heads at once)
+        (or every head by its own root mean square, without a weight)
+    q <- q * temperature(position), where there is one
     the first `rotary_dim` numbers of every head of q and k turned by the position
     s_ij = q_i . k_j * scale  for  j <= i  and  (i - j < window  or  j < keep_first)
     a_i = sum_j exp(s_ij) v_j / (sum_j exp(s_ij) + exp(sink[h]))
-    out = Wo [out_scale * a]
+    out = Wo [out_scale * a * sigmoid(h Wg^T)]         (the gate, element by element, if there is one)
 
 The fused projection leaves fp32 (its accumulator, unrounded); the two norms, the rotation and
 the cache write are one kernel (`csrc/qk_prepare.cu`); scores, softmax weights, the sink and the
@@ -37,24 +39,26 @@ class WindowSinkAttention(Part):
             raise ValueError(f"{s.heads} heads are not a multiple of {s.kv_heads} kv heads")
         if s.head_dim > 640 or s.value_dim > 512:
             raise ValueError("the attention kernel takes head_dim up to 640 and value_dim up to 512")
-        if s.qk_norm not in (None, "whole"):
-            raise ValueError(f"qk_norm {s.qk_norm!r}: only 'whole' (or None) is built")
+        if s.qk_norm not in (None, "whole", "head"):
+            raise ValueError(f"qk_norm {s.qk_norm!r}: 'whole', 'head' and None are built")
         if s.keep_first and not s.window:
             raise ValueError("keep_first goes with a window")
         self.q_cols = s.heads * s.head_dim
         self.k_cols = s.kv_heads * s.head_dim
         self.v_cols = s.kv_heads * s.value_dim
         self.position = None if s.position is None else build_part(s.position, prefix, mode)
-        self.sink = None
+        self.sink = self.temperature = None
+        self.g_cols = s.heads * s.value_dim if s.gate else 0
 
     # -- what a branch offers -------------------------------------------------------------
 
     @property
     def input_rows(self) -> int:
-        return self.q_cols + self.k_cols + self.v_cols
+        return self.q_cols + self.k_cols + self.v_cols + self.g_cols
 
     def _inputs(self):
-        return (("q", self.q_cols), ("k", self.k_cols), ("v", self.v_cols))
+        rows = (("q", self.q_cols), ("k", self.k_cols), ("v", self.v_cols))
+        return rows + (("g", self.g_cols),) if self.g_cols else rows
 
     def input_decls(self, group):
         """The matrices that read the mixer's input, in the order of their rows in the fused
@@ -67,8 +71,8 @@ class WindowSinkAttention(Part):
         decls = []
         if s.bias:
             decls += [TensorDecl(f"{p}{n}.b", (rows,), group=p + "fused.b")
-                      for n, rows in self._inputs()]
-        if s.qk_norm:
+                      for n, rows in self._inputs() if n != "g"]
+        if s.qk_norm == "whole":
             decls += [TensorDecl(p + "q.norm", (self.q_cols,), init="ones_normal"),
                       TensorDecl(p + "k.norm", (self.k_cols,), init="ones_normal")]
         if s.sink:
@@ -83,13 +87,15 @@ class WindowSinkAttention(Part):
         p = self.prefix
         b = arena.group_view(p + "fused.b")
         if b is None:
-            b = torch.cat([arena.view(f"{p}{n}.b") for n, _ in self._inputs()])
+            b = torch.cat([arena.view(f"{p}{n}.b") for n, _ in self._inputs() if n != "g"])
+        if self.g_cols:                        # (the gate has no bias)
+            b = torch.cat([b, torch.zeros(self.g_cols, dtype=b.dtype, device=b.device)])
         return b
 
     def bind_rest(self, arena):
         s, p = self.spec, self.prefix
-        self.wq = arena.view(p + "q.norm") if s.qk_norm else None
-        self.wk = arena.view(p + "k.norm") if s.qk_norm else None
+        self.wq = arena.view(p + "q.norm") if s.qk_norm == "whole" else None
+        self.wk = arena.view(p + "k.norm") if s.qk_norm == "whole" else None
         self.sink = arena.view(p + "sink").float().contiguous() if s.sink else None
         self.w_o = arena.view(p + "o")
 
@@ -107,12 +113,21 @@ class WindowSinkAttention(Part):
         q = ops.qk_prepare(proj, offset, offset + self.q_cols, offset + self.q_cols + self.k_cols,
                            s.heads, s.kv_heads, s.head_dim, s.value_dim, self.wq, self.wk, s.eps,
                            cos, sin, step.positions, step.token_seq, view.block_table, view.keys,
-                           view.values, self.act_dtype, write_cache)
+                           view.values, self.act_dtype, write_cache, norm=s.qk_norm,
+                           temperature=self._temperature(step))
+        g_off = offset + self.q_cols + self.k_cols + self.v_cols
+        gate = proj[:, g_off:g_off + self.g_cols] if self.g_cols else None
         return ops.cached_attention(
             q.view(q.shape[0], s.heads, s.head_dim), view.keys, view.values, step.positions,
             step.token_seq, view.block_table, s.heads, s.head_dim, s.value_dim, s.scale,
             window=s.window, keep_first=s.keep_first if s.window else 0, sink=self.sink,
-            out_scale=s.out_scale, **self._decode_form(step)).view(q.shape[0], -1)
+            out_scale=s.out_scale, elem_gate=gate, **self._decode_form(step)).view(q.shape[0], -1)
+
+    def _temperature(self, step):
+        if self.temperature is not None and step.max_position >= self.temperature.numel():
+            raise ValueError(f"position {step.max_position} is beyond the table of "
+                             f"{self.temperature.numel()} query temperatures")
+        return self.temperature
 
     def _decode_form(self, step) -> dict:
         """For decode steps in bfloat16 a block's warps are one token's groups of heads and
@@ -144,6 +159,11 @@ class WindowSinkAttention(Part):
     def prepare(self, device, max_positions):
         if self.position is not None:
             self.position.prepare(device, max_positions)
+        t = self.spec.q_temp
+        if t is not None:       # worked out in float64, kept in fp32
+            p = torch.arange(max_positions, dtype=torch.float64)
+            self.temperature = (1.0 + t.coef * torch.log(torch.floor((p + 1.0) / t.every) + 1.0)
+                                ).to(device=device, dtype=torch.float32)
 
     def cache_need(self):
         s = self.spec
