@@ -14,7 +14,6 @@ import plain_felovik as plain
 import semantic_aware_adaptive_kv_cache_precision_b200 as sakv
 from helpers import assert_same_logits
 from felovik_configs import dense, layer, moe
-from gesuvik_configs import rows_agree
 
 pytestmark = pytest.mark.gpu
 
@@ -63,6 +62,22 @@ def draw(seed, all_chosen=False):
             "layers": layers}
 
 
+def row_errors(got, want):
+    """Each row's largest difference over its spread."""
+    return np.abs(np.asarray(got, dtype=np.float64) - want).max(axis=-1) / want.std(axis=-1)
+
+
+def conditioning(cfg, tensors, p, want):
+    """How a drawn model answers rounding, from the plain model alone: the median row's
+    difference when every weight moves by up to 2^-8 of itself, over 0.05 (what it is for most
+    draws or less), 1 at least. Some draws divide small sums by their root mean square layer after
+    layer and answer ten times as strongly."""
+    rng = np.random.default_rng(1)
+    moved = {k: np.asarray(v, dtype=np.float64) * (1 + rng.uniform(-1, 1, np.shape(v)) * 2.0 ** -8)
+             for k, v in tensors.items()}
+    return max(1.0, np.median(row_errors(plain.forward(cfg, moved, p), want)) / 0.05)
+
+
 @pytest.mark.parametrize("seed", range(24))
 def test_a_drawn_configuration_in_32_bits(seed, tmp_path):
     config = draw(seed)
@@ -73,7 +88,10 @@ def test_a_drawn_configuration_in_32_bits(seed, tmp_path):
     prompts = [rng.integers(0, config["vocab"], n).astype(np.int64) for n in (170, 37, 2)]
     whole = [engine.forward(p) for p in prompts]
     for got, p in zip(whole, prompts):
-        rows_agree(got, plain.forward(cfg, tensors, p), "float32", f"seed {seed}")
+        want = plain.forward(cfg, tensors, p)
+        err, answer = row_errors(got, want), conditioning(cfg, tensors, p, want)
+        assert np.quantile(err, 0.97) <= 5e-5 * answer and err.max() <= 2e-3 * answer, \
+            f"seed {seed}: worst row {err.max():.2e}, 97 of 100 within {np.quantile(err, 0.97):.2e}"
     # the longest prompt again: most of it in one step, its last 40 tokens one by one
     p = prompts[0]
     (slot,) = engine.open(1)
@@ -110,8 +128,7 @@ def test_a_drawn_configuration_in_32_bits(seed, tmp_path):
 def test_a_drawn_configuration_in_16_bits(seed, tmp_path):
     """A prompt long enough for the recurrence to walk it in runs, then tokens one by one; every
     expert chosen for every token (a choice that rounding turns is no fault); judged by the
-    median row within a tenth of its spread, since a drawn configuration may be badly
-    conditioned."""
+    median row, within a tenth of its spread where the model is well conditioned."""
     config = draw(seed, all_chosen=True)
     folder = sakv.write_random_model(tmp_path / "m", copy.deepcopy(config), seed, dtype="bfloat16")
     cfg, tensors = plain.read_model_folder(folder)
@@ -125,7 +142,7 @@ def test_a_drawn_configuration_in_16_bits(seed, tmp_path):
     engine.close([slot])
     got = np.concatenate(rows)
     assert np.isfinite(got).all()
-    worst = np.abs(got - want).max(axis=-1) / want.std(axis=-1)
-    assert np.median(worst[:290]) <= 0.1, f"seed {seed}: the prompt's median row {np.median(worst[:290]):.3f}"
-    assert np.median(worst[290:]) <= 0.1, f"seed {seed}: the decoded median row {np.median(worst[290:]):.3f}"
+    err, answer = row_errors(got, want), conditioning(cfg, tensors, p, want)
+    for what, rows in (("prompt", err[:290]), ("decoded tokens", err[290:])):
+        assert np.median(rows) <= 0.1 * answer, f"seed {seed}: the {what}'s median row {np.median(rows):.3f}"
     assert engine.graph_failure is None
