@@ -380,6 +380,21 @@ def kernel_case(name: str) -> int:
         run = lambda i: ops.decay_attention(proj, 0, heads * dim, 2 * heads * dim, heads, dim, vdim,
                                             less_one, state, step, run=64, activation=False,
                                             cos=cos, sin=sin, key_scale=dim ** -0.5)
+    elif name == "dual_scan_4096":
+        # the state-space dual scan over one prompt of 4,096 tokens at the `2k` size of `--design
+        # felovik` (64 heads of 128 x 64, one group of B and C), walked in runs of 64 tokens:
+        # about 270 MB, most of it the runs' states
+        from types import SimpleNamespace
+        n, heads, vdim, ns = 4096, 64, 64, 128
+        xbc = torch.randn(n, heads * vdim + 2 * ns, device=dev).to(torch.bfloat16)
+        dt = torch.randn(n, heads, device=dev)
+        bias, a = torch.full((heads,), -3.0, device=dev), -torch.rand(heads, device=dev) - 0.1
+        skip = torch.ones(heads, device=dev)
+        state = torch.zeros(1, heads, vdim, ns, device=dev)
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        step = SimpleNamespace(cu_seqlens=i32([0, n]), slots=i32([0]), sequences=1, max_new=n)
+        run = lambda i: ops.dual_scan(xbc, 0, heads * vdim, heads * vdim + ns, dt, bias, a, skip,
+                                      heads, 1, ns, vdim, state, step, run=64)
     else:
         raise SystemExit(f"unknown kernel case {name}")
     for i in range(4):
@@ -700,6 +715,117 @@ def zodirax_rates(size, zt, tt, batch, context, tokens, hbm) -> dict:
     return out
 
 
+#: layer sizes for `--design felovik`: (width; attention heads / kv heads x (dim, vdim); the
+#: recurrence's heads, vdim, state, groups, taps and norm parts; dense feed-forward; experts,
+#: chosen, their width, groups of experts and how many stay open)
+FELOVIK_SIZES = {
+    "1k": dict(width=1024, attention=(8, 2, 128, 128), dual=(32, 64, 128, 1, 4, 1), ff=4096,
+               experts=(16, 2, 1024, 4, 2), vocab=32768, layers=6),
+    "2k": dict(width=2048, attention=(16, 4, 128, 128), dual=(64, 64, 128, 1, 4, 1), ff=8192,
+               experts=(32, 4, 1024, 8, 4), vocab=32768, layers=6),
+}
+
+
+def felovik_configs(size: dict) -> dict:
+    """Configs by label: Felovik with dense feed-forwards only and with experts in two layers of
+    three, and the Zodirax config whose every layer is the same pair (attention of equal heads
+    without a window beside a fading state of equal heads and sizes) with a dense feed-forward
+    of equal size: the library's other design with two mixers side by side."""
+    heads, kv_heads, dim, vdim = size["attention"]
+    dheads, dvdim, state, groups, taps, parts = size["dual"]
+    experts, top, eff, count, keep = size["experts"]
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5}
+    mixer = {"left": dict(left, q_temp={"coef": 0.1, "every": 1024}),
+             "right": {"heads": dheads, "vdim": dvdim, "state": state, "groups": groups,
+                       "conv": taps, "norm_groups": parts}}
+    dense = {"kind": "dense", "ff": size["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": eff},
+           "router": {"experts": experts, "top": top, "groups": {"count": count, "keep": keep}}}
+
+    def felovik(mlps):
+        return {"architecture": "Felovik", "vocab": size["vocab"], "width": size["width"],
+                "max_positions": 16384, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+                "postln_alpha": 2.0, "initializer_range": 0.02,
+                "layers": [{"type": "parallel", "mixer": mixer, "mlp": m} for m in mlps]}
+
+    fading = {"heads": dheads, "dim": state, "vdim": dvdim,
+              "decay": [1.0 - 2.0 ** -(2 + 8 * h / dheads) for h in range(dheads)]}
+    zodirax = {"architecture": "Zodirax", "vocab": size["vocab"], "width": size["width"],
+               "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "initializer_range": 0.02,
+               "layers": [{"type": "parallel", "mlp": {"kind": "dense", "ff": size["ff"]},
+                           "mixer": {"left": left, "right": fading, "left_scale": 1.0,
+                                     "right_scale": 1.0}}] * size["layers"]}
+    return {"zodirax": zodirax, "felovik_dense": felovik([dense] * size["layers"]),
+            "felovik_experts": felovik([dense if i % 3 == 0 else moe
+                                        for i in range(size["layers"])])}
+
+
+def felovik_rates(size, kernels, gsize, batch, context, tokens, hbm) -> dict:
+    """What the designs' own kernels must move or compute in the timed steps, against the
+    measured peaks. `kernels`: kernel times by label (`felovik_configs`, and `gesuvik` of sizes
+    `gsize` for the experts)."""
+    heads, kv_heads, dim, vdim = size["attention"]
+    dheads, dvdim, state, groups, taps, parts = size["dual"]
+    experts, top, eff, _, _ = size["experts"]
+    n, width = size["layers"], size["width"]
+    n_moe = sum(1 for i in range(n) if i % 3)
+    inner = dheads * dvdim
+    channels = inner + 2 * groups * state
+    f, e, z, g = (kernels[k] for k in ("felovik_dense", "felovik_experts", "zodirax", "gesuvik"))
+
+    def of_hbm(nbytes, us):
+        return round(nbytes / (us * 1e-6) / 1e9 / hbm, 3) if us else None
+
+    def tflops(flops, us):
+        return round(flops / (us * 1e-6) / 1e12, 2) if us else None
+
+    out = {}
+    # the recurrence over a prompt: a state element's decay, input and output a token; bytes: x, B
+    # and C (bf16) and the step sizes in, y (fp32) out. Zodirax: q, k, v and o a head, fp32
+    ops_ = 6.0 * tokens * dheads * state * dvdim * n
+    out["dual_scan_prefill_tflops_fp32"] = tflops(ops_, f["prefill"].get("dual_scan"))
+    out["zodirax_fading_prefill_tflops_fp32"] = tflops(ops_, z["prefill"].get("decay_attention"))
+    out["dual_scan_prefill_of_measured_hbm"] = of_hbm(
+        tokens * (channels * 2 + dheads * 4 + inner * 4) * n, f["prefill"].get("dual_scan"))
+    out["zodirax_fading_prefill_of_measured_hbm"] = of_hbm(
+        tokens * dheads * (2 * state + 2 * dvdim) * 4 * n, z["prefill"].get("decay_attention"))
+    moved = batch * dheads * state * dvdim * 4 * 2 * n                 # the state, in and out
+    out["dual_scan_decode_of_measured_hbm"] = of_hbm(moved, f["decode"].get("dual_scan"))
+    out["zodirax_fading_decode_of_measured_hbm"] = of_hbm(moved, z["decode"].get("decay_attention"))
+    flops = 2.0 * heads * (dim + vdim) * tokens * (tokens + 1) / 2 * n
+    read = batch * context * kv_heads * (dim + vdim) * 2 * n
+    for label, t in (("", f), ("zodirax_", z)):
+        out[label + "attention_prefill_tflops_fp32"] = tflops(flops, t["prefill"].get("cached_attention"))
+        out[label + "attention_decode_of_measured_hbm"] = of_hbm(read, t["decode"].get("cached_attention"))
+        qkv = heads * dim + kv_heads * (dim + vdim)
+        out[label + "qk_prepare_prefill_of_measured_hbm"] = of_hbm(
+            tokens * qkv * 6 * n, t["prefill"].get("qk_prepare"))
+    # the step between two sublayers: x and y (two ys after the mixer) in, x and its bf16 copy out
+    out["rms_join_prefill_of_measured_hbm"] = of_hbm(
+        tokens * width * (4 * 3 + 2 + 2) * 2 * n, f["prefill"].get("rms_join"))
+    out["zodirax_rms_update_prefill_of_measured_hbm"] = of_hbm(
+        tokens * width * (4 * 3 + 2) * 2 * n, z["prefill"].get("rms_update"))
+    # the gated norm: y (and the gate) in, bf16 out
+    for label, t in (("", f), ("zodirax_", z)):
+        out[label + "norm_gate_prefill_of_measured_hbm"] = of_hbm(
+            tokens * inner * 10 * n, t["prefill"].get("norm_gate"))
+    out["conv_prefill_of_measured_hbm"] = of_hbm(tokens * channels * 6 * n,
+                                                 f["prefill"].get("causal_conv"))
+    # dense feed-forward, gate and up with the activation (the kernel of each that makes it)
+    flops = 4.0 * tokens * width * size["ff"] * n
+    for label, t in (("", f), ("zodirax_", z)):
+        out[label + "gated_product_prefill_tflops_bf16"] = tflops(flops, t["prefill"].get("gemm_pair"))
+    for label, t, top_, eff_, layers, real in (
+            ("", e, top, eff, n_moe, 1.0),
+            ("gesuvik_", g, gsize["experts"][2], gsize["experts"][3], gsize["layers"],
+             gsize["experts"][0] / (gsize["experts"][0] + gsize["experts"][1]))):
+        out[label + "experts_prefill_tflops_bf16"] = tflops(
+            6.0 * tokens * top_ * real * eff_ * width * layers, t["prefill"].get("moe_product"))
+        out[label + "experts_decode_of_measured_hbm"] = of_hbm(
+            min(batch * top_, experts) * 3 * eff_ * width * 2 * layers, t["decode"].get("moe_product"))
+    return out
+
+
 def design_configs(size: dict) -> tuple:
     """(Tebonex config, the Qwen2 config of equal width, depth, heads and feed-forward)."""
     heads, kv_heads, dim = size["attention"]
@@ -880,6 +1006,35 @@ def design_arm(args) -> int:
                           "batch": batch, "context": context, "prefill_tokens": tokens, "steps": K,
                           "warmup": W, "peaks": pk, "sizes": rows}))
         return 0
+    if args.design == "felovik":
+        for name in sizes:
+            size, gsize = FELOVIK_SIZES[name], GESUVIK_SIZES[name]
+            row = {"size": name, **{k: size[k] for k in ("width", "layers", "ff", "attention",
+                                                         "dual", "experts")}}
+            kernels = {}
+            configs = dict(felovik_configs(size), gesuvik=gesuvik_configs(gsize))
+            for label, config in configs.items():
+                engine, slots, prompt, out = measure(config)
+                row[label] = out
+                engine.close(slots)
+                engine.release()
+                del engine
+                torch.cuda.empty_cache()
+                engine, slots, prompt, _ = measure(config, graphs=False)
+                row[label + "_kernels_us"] = kernels[label] = kernel_times(engine, slots, prompt)
+                engine.close(slots)
+                engine.release()
+                del engine
+                torch.cuda.empty_cache()
+            row["kernel_rates"] = felovik_rates(size, kernels, gsize, batch, context, tokens, hbm)
+            rows.append(row)
+        print(json.dumps({"design": "felovik", "beside": "zodirax of equal width, depth, attention "
+                          "heads, recurrent state and feed-forward size, every layer two mixers "
+                          "side by side; gesuvik for the experts", "dtype": "bf16",
+                          "data": "synthetic (random weights and tokens; weights larger than L2)",
+                          "batch": batch, "context": context, "prefill_tokens": tokens, "steps": K,
+                          "warmup": W, "peaks": pk, "sizes": rows}))
+        return 0
     if args.design == "zodirax":
         for name in sizes:
             size = ZODIRAX_SIZES[name]
@@ -965,14 +1120,14 @@ def design_arm(args) -> int:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=["tebonex", "venanex", "zodirax", "gesuvik"],
+    ap.add_argument("--design", default=None, choices=["tebonex", "venanex", "zodirax", "gesuvik", "felovik"],
                     help="instead of the default workload: the named design at layer sizes "
                          "that resemble real models, beside the Qwen2 decoder of equal size")
     ap.add_argument("--design-sizes", default="1k,2k", help="which of: " + ", ".join(DESIGN_SIZES))
     ap.add_argument("--kernel", default=None,
                     help="run one kernel case for a profiler: gemm_gateup_b8, gemm_down_b8, "
                          "gemm_head_b8, gemm_gated_2048, selective_scan_4096, retention_4096, "
-                         "attention_decode_b64, attention_prefill_2048")
+                         "dual_scan_4096, attention_decode_b64, attention_prefill_2048")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=3)
