@@ -482,6 +482,11 @@ __global__ void decay_carry_kernel(const float* __restrict__ decay_less_one,
 // here from the projection's column, which multiplies x and chooses the token's decay, and D x
 // added to the output. State in memory: [slots, heads, vdim, dim] (a column's rows together).
 // PHASE as above; a run's decay to the carry kernel is the sum of its step sizes.
+//
+// CV neighbouring columns belong to one thread (4 where the step's walks fill the GPU, else 1):
+// what a token brings for a lane's rows is read once for all of them, and with four the sums
+// over the lanes are exchanged half by half, so that each lane ends with one column. The pairs
+// that are added are the same either way, and so is every sum.
 // ---------------------------------------------------------------------------------------
 template <typename C>
 struct DualScan {
@@ -502,8 +507,8 @@ struct DualScan {
   float* dt_sums;                  // [sequences, max_chunks, heads]
 };
 
-template <int RP, int PHASE, typename C>
-__global__ void dual_scan_kernel(const DualScan<C> p) {
+template <int RP, int CV, int PHASE, typename C>
+__global__ void __launch_bounds__(256) dual_scan_kernel(const DualScan<C> p) {
   extern __shared__ __align__(16) float shared[];
   const int padded = p.rs * RP;                     // dim rounded up to whole lanes
   const int padded_shift = 31 - __clz(padded);
@@ -522,28 +527,36 @@ __global__ void dual_scan_kernel(const DualScan<C> p) {
   }
   const int h = blockIdx.y, col0 = blockIdx.x * p.cols;
   const int group_off = h / (p.heads / p.groups) * p.dim;
-  const int r = threadIdx.x % p.rs, j = threadIdx.x / p.rs;
-  const int col = col0 + j, dim = p.dim;
-  const bool live = col < p.vdim;
+  const int r = threadIdx.x % p.rs, j = threadIdx.x / p.rs * CV;
+  const int col = col0 + j, dim = p.dim;            // this thread's first column
   const float a = p.a[h], bias = p.dt_bias[h], skip = p.d_skip[h];
-  float s[RP];
+  float s[CV][RP];
   const long long per_seq = (long long)p.heads * p.vdim * dim;
-  const long long place = ((long long)h * p.vdim + (live ? col : 0)) * dim + r * RP;
+  const long long place = ((long long)h * p.vdim + col) * dim + r * RP;    // (used while col < vdim)
   float* mine = PHASE == 0 ? p.state + p.slots[b] * per_seq + place
                            : p.scratch + ((long long)b * p.max_chunks + piece) * per_seq + place;
   const bool wide = dim % 4 == 0;                   // (then every lane's rows are 16-byte aligned)
 #pragma unroll
-  for (int k = 0; k < RP; k += 4) {
-    const int at = r * RP + k;
-    if (PHASE != 1 && live && wide && at < dim) {
-      const float4 v = *reinterpret_cast<const float4*>(mine + k);
-      s[k] = v.x; s[k + 1] = v.y; s[k + 2] = v.z; s[k + 3] = v.w;
-    } else {
+  for (int c = 0; c < CV; ++c) {
+    const bool live = col + c < p.vdim;
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-        s[k + i] = (PHASE != 1 && live && at + i < dim) ? mine[k + i] : 0.f;
+    for (int k = 0; k < RP; k += 4) {
+      const int at = r * RP + k;
+      if (PHASE != 1 && live && wide && at < dim) {
+        const float4 v = *reinterpret_cast<const float4*>(mine + (long long)c * dim + k);
+        s[c][k] = v.x; s[c][k + 1] = v.y; s[c][k + 2] = v.z; s[c][k + 3] = v.w;
+      } else {
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          s[c][k + i] = (PHASE != 1 && live && at + i < dim) ? mine[(long long)c * dim + k + i] : 0.f;
+      }
     }
   }
+  // the column whose output this lane writes (none: -1): lane 0's only one, or with four columns
+  // the one that the exchange below leaves with the lane
+  int own = r == 0 ? 0 : -1;
+  if (CV == 4) own = (r & (p.rs / 4 - 1)) == 0 ? r / (p.rs / 4) : -1;
+  if (own >= 0 && col + own >= p.vdim) own = -1;
   float dt_sum = 0.f;
   for (int t0 = first; t0 < last; t0 += kRun) {
     const int run = last - t0 < kRun ? last - t0 : kRun;
@@ -567,45 +580,78 @@ __global__ void dual_scan_kernel(const DualScan<C> p) {
     }
     __syncthreads();
     for (int tt = 0; tt < run; ++tt) {
-      const float x = vs[tt * p.cols + j], dt = steps[tt], fade = fades[tt];
-      const float v = dt * x;
+      const float* xs = vs + tt * p.cols + j;
+      const float dt = steps[tt], fade = fades[tt];
+      float v[CV], o[CV];
+      if constexpr (CV == 4) {
+        const float4 x4 = *reinterpret_cast<const float4*>(xs);
+        v[0] = dt * x4.x; v[1] = dt * x4.y; v[2] = dt * x4.z; v[3] = dt * x4.w;
+      } else {
+        v[0] = dt * xs[0];
+      }
+#pragma unroll
+      for (int c = 0; c < CV; ++c) o[c] = 0.f;
       dt_sum += dt;
-      float o = 0.f;
       const float4* k4 = reinterpret_cast<const float4*>(ks + tt * padded + r * RP);
       const float4* q4 = reinterpret_cast<const float4*>(qs + tt * padded + r * RP);
 #pragma unroll
       for (int k = 0; k < RP; k += 4) {
         const float4 kk = k4[k >> 2];
-        // S + (e^(dt A) - 1) S + dt B x: a decay close to 1 keeps its distance from 1
-        s[k] = fmaf(kk.x, v, fmaf(fade, s[k], s[k]));
-        s[k + 1] = fmaf(kk.y, v, fmaf(fade, s[k + 1], s[k + 1]));
-        s[k + 2] = fmaf(kk.z, v, fmaf(fade, s[k + 2], s[k + 2]));
-        s[k + 3] = fmaf(kk.w, v, fmaf(fade, s[k + 3], s[k + 3]));
-        if (PHASE != 1) {
-          const float4 qq = q4[k >> 2];
-          o = fmaf(s[k], qq.x, o);
-          o = fmaf(s[k + 1], qq.y, o);
-          o = fmaf(s[k + 2], qq.z, o);
-          o = fmaf(s[k + 3], qq.w, o);
+        const float4 qq = PHASE != 1 ? q4[k >> 2] : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int c = 0; c < CV; ++c) {
+          // S + (e^(dt A) - 1) S + dt B x: a decay close to 1 keeps its distance from 1
+          float* sc = s[c] + k;
+          sc[0] = fmaf(kk.x, v[c], fmaf(fade, sc[0], sc[0]));
+          sc[1] = fmaf(kk.y, v[c], fmaf(fade, sc[1], sc[1]));
+          sc[2] = fmaf(kk.z, v[c], fmaf(fade, sc[2], sc[2]));
+          sc[3] = fmaf(kk.w, v[c], fmaf(fade, sc[3], sc[3]));
+          if (PHASE != 1) {
+            o[c] = fmaf(sc[0], qq.x, o[c]);
+            o[c] = fmaf(sc[1], qq.y, o[c]);
+            o[c] = fmaf(sc[2], qq.z, o[c]);
+            o[c] = fmaf(sc[3], qq.w, o[c]);
+          }
         }
       }
       if (PHASE != 1) {
-        for (int d = p.rs >> 1; d > 0; d >>= 1) o += __shfl_xor_sync(0xffffffffu, o, d);
-        if (r == 0 && live)
-          p.out[((long long)(t0 + tt) * p.heads + h) * p.vdim + col] = fmaf(skip, x, o);
+        float sum;
+        int d = p.rs >> 1;
+        if constexpr (CV == 4) {                       // (rs >= 4)
+          const bool up = r & d;                       // columns 2, 3 stay with the upper half
+          float a0 = up ? o[2] : o[0], a1 = up ? o[3] : o[1];
+          a0 += __shfl_xor_sync(0xffffffffu, up ? o[0] : o[2], d);
+          a1 += __shfl_xor_sync(0xffffffffu, up ? o[1] : o[3], d);
+          d >>= 1;
+          const bool odd = r & d;
+          sum = (odd ? a1 : a0) + __shfl_xor_sync(0xffffffffu, odd ? a0 : a1, d);
+          d >>= 1;
+        } else {
+          sum = o[0];
+        }
+        for (; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+        if (own >= 0)
+          p.out[((long long)(t0 + tt) * p.heads + h) * p.vdim + col + own] =
+              fmaf(skip, xs[own], sum);
       }
     }
   }
-  if (live && (PHASE == 1 || (PHASE == 0 && p.keep_state))) {
+  if (PHASE == 1 || (PHASE == 0 && p.keep_state)) {
 #pragma unroll
-    for (int k = 0; k < RP; k += 4) {
-      const int at = r * RP + k;
-      if (wide && at < dim) {
-        *reinterpret_cast<float4*>(mine + k) = make_float4(s[k], s[k + 1], s[k + 2], s[k + 3]);
-      } else {
+    for (int c = 0; c < CV; ++c) {
+      if (col + c >= p.vdim) continue;
+      float* to = mine + (long long)c * dim;
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
-          if (at + i < dim) mine[k + i] = s[k + i];
+      for (int k = 0; k < RP; k += 4) {
+        const int at = r * RP + k;
+        if (wide && at < dim) {
+          *reinterpret_cast<float4*>(to + k) =
+              make_float4(s[c][k], s[c][k + 1], s[c][k + 2], s[c][k + 3]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            if (at + i < dim) to[k + i] = s[c][k + i];
+        }
       }
     }
   }
@@ -925,18 +971,27 @@ SAKV_EXPORT int sakv_dual_scan(const void* xbc, int c_dtype, long long stride, i
   const long long walks = runs ? (long long)sequences * max_chunks : sequences;
   const int rp = dim < 128 ? 4 : 8;        // (rows a lane; 16 lanes a column from 128 rows on)
   const int rs = lanes_for(dim, rp);
-  int cols = 256 / rs;                       // value columns a block
-  while (cols > 1 && (long long)((vdim + cols - 1) / cols) * heads * walks < 2LL * sm_count())
-    cols /= 2;
-  while (cols > 1 && cols / 2 >= vdim) cols /= 2;
-  if (cols * rs < 32) cols = 32 / rs;        // whole warps
+  // four columns a thread where the step's blocks then still fill the GPU (a prompt's runs)
+  const bool four = rs >= 4 && vdim >= 4 &&
+                    (long long)((vdim + 1024 / rs - 1) / (1024 / rs)) * heads * walks >= 2LL * sm_count();
+  const int cv = four ? 4 : 1;
+  int lanes_across = 256 / rs;               // threads of a block side by side over the columns
+  while (lanes_across > 1 &&
+         (long long)((vdim + lanes_across * cv - 1) / (lanes_across * cv)) * heads * walks <
+             2LL * sm_count())
+    lanes_across /= 2;
+  while (lanes_across > 1 && lanes_across / 2 * cv >= vdim) lanes_across /= 2;
+  if (lanes_across * rs < 32) lanes_across = 32 / rs;        // whole warps
+  const int cols = lanes_across * cv;        // value columns a block
   const dim3 grid((unsigned)((vdim + cols - 1) / cols), (unsigned)heads, (unsigned)walks);
   const size_t smem = (size_t)kRun * (2 * rs * rp + cols + 2) * sizeof(float);
-#define SAKV_DUAL(RP, PHASE, C)                                                                  \
-  launch_ordered(dual_scan_kernel<RP, PHASE, C>, grid, dim3(cols * rs), smem, stream,            \
+#define SAKV_DUAL_CV(RP, CV, PHASE, C)                                                           \
+  launch_ordered(dual_scan_kernel<RP, CV, PHASE, C>, grid, dim3(lanes_across * rs), smem, stream, \
                  DualScan<C>{(const C*)xbc, stride, x_off, b_off, c_off, dt, dt_stride, dt_bias, \
                              a, d_skip, state, cu_seqlens, slots, out, heads, groups, dim, vdim, \
                              rs, cols, keep_state, chunk_len, max_chunks, scratch, dt_sums})
+#define SAKV_DUAL(RP, PHASE, C)                                                                  \
+  (four ? SAKV_DUAL_CV(RP, 4, PHASE, C) : SAKV_DUAL_CV(RP, 1, PHASE, C))
 #define SAKV_DUAL_ALL(RP, C)                                                                     \
   do {                                                                                           \
     if (!runs) return SAKV_DUAL(RP, 0, C);                                                       \
@@ -960,6 +1015,7 @@ SAKV_EXPORT int sakv_dual_scan(const void* xbc, int c_dtype, long long stride, i
   }
 #undef SAKV_DUAL_ALL
 #undef SAKV_DUAL
+#undef SAKV_DUAL_CV
   return cudaErrorInvalidValue;
 }
 

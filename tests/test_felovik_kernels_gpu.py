@@ -194,7 +194,7 @@ def test_keys_far_back_and_at_block_borders_with_an_elementwise_gate(dtype, head
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("heads,vdim,state,groups", [
     (4, 16, 24, 2), (3, 24, 16, 1), (5, 12, 7, 5), (3, 10, 1, 1), (6, 8, 40, 3), (2, 64, 160, 2),
-    (4, 64, 128, 1), (1, 36, 36, 1), (2, 3, 200, 1)])
+    (4, 64, 128, 1), (1, 36, 36, 1), (2, 3, 200, 1), (8, 10, 24, 2), (7, 70, 64, 1)])
 def test_dual_scan_over_pieces_with_a_token_far_back(dtype, heads, vdim, state, groups):
     """Head 0 hardly fades and is fed once, at token 2, far more than anything after it; the last
     token's C reads exactly that. Other heads fade within a token or two. Pieces down to one
@@ -258,6 +258,32 @@ def test_dual_scan_over_pieces_with_a_token_far_back(dtype, heads, vdim, state, 
                   dev(a), dev(d_skip), heads, groups, state, vdim, st, scan_step([5], [0]),
                   keep_state=False, run=2)
     assert torch.equal(st, before)
+
+
+@pytest.mark.parametrize("heads,vdim,state,groups", [(6, 24, 40, 2), (4, 70, 128, 1), (8, 9, 16, 8)])
+def test_a_full_step_and_single_sequences_give_the_same_bits(heads, vdim, state, groups):
+    """Ninety sequences fill the GPU (several columns a thread), one does not (one column a
+    thread): every output and state is the same to the bit."""
+    g = torch.Generator(device=DEV).manual_seed(heads)
+    lengths = [1 + 7 * i % 40 for i in range(90)]
+    n, inner, gn = sum(lengths), heads * vdim, groups * state
+    rand = lambda *shape: torch.randn(shape, generator=g, device=DEV)
+    xbc, dt = rand(n, inner + 2 * gn), rand(n, heads)
+    bias, a, skip = rand(heads) - 2.0, -torch.exp(rand(heads)), rand(heads)
+
+    def run(x, d, lengths, slots, state_t):
+        return ops.dual_scan(x, 0, inner, inner + gn, d, bias, a, skip, heads, groups, state, vdim,
+                             state_t, scan_step(lengths, slots))
+
+    together = torch.zeros((90, heads, vdim, state), device=DEV)
+    out = run(xbc, dt, lengths, list(range(90)), together)
+    at = 0
+    for i, m in enumerate(lengths):
+        if i % 9 == 0:
+            alone = torch.zeros((1, heads, vdim, state), device=DEV)
+            got = run(xbc[at:at + m], dt[at:at + m], [m], [0], alone)
+            assert torch.equal(got, out[at:at + m]) and torch.equal(alone[0], together[i])
+        at += m
 
 
 def test_the_convolution_reads_columns_inside_a_wider_projection():
