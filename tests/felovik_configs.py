@@ -61,6 +61,6 @@ WIDE = {"architecture": "Felovik", "vocab": 97, "width": 128, "max_positions": 1
                          dense(256, 7.0)),
                    layer((2, 2, 64, 320, 0.125, (0.6, 200)), (2, 64, 160, 2, 4, 2),
                          moe(16, 4, 128, (8, 3))),
-                   layer((8, 2, 64, 64, 0.125, None), (8, 32, 64, 4, 4, 8),
+                   layer((6, 2, 64, 48, 0.15, None), (8, 32, 64, 4, 4, 8),
                          moe(4, 4, 32, (2, 2)))]}
 CONFIGS = {"mixed": (MIXED, 51), "odd": (ODD, 52), "wide": (WIDE, 53)}

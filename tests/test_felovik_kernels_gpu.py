@@ -326,7 +326,7 @@ def test_the_gate_comes_before_a_norm_in_parts(dtype, width, parts):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("n,width,experts,top,ff,groups", [
-    (77, 96, 8, 3, 48, (4, 2)), (1, 64, 12, 4, 40, (3, 2)), (200, 64, 36, 6, 24, (6, 3)),
+    (77, 96, 8, 3, 48, (4, 2)), (1, 64, 10, 4, 40, (5, 3)), (200, 64, 36, 6, 24, (6, 3)),
     (33, 100, 9, 1, 22, (9, 2)), (5, 72, 6, 4, 50, (3, 2)), (300, 128, 128, 8, 16, (64, 5)),
     (90, 64, 5, 2, 130, None), (70, 48, 4, 4, 32, (2, 2)), (150, 64, 80, 3, 16, (2, 1)),
     (64, 64, 80, 5, 16, (40, 7))])
