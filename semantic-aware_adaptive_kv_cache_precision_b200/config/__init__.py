@@ -1,7 +1,7 @@
 """Typed configurations and the architecture registry."""
 
-from .specs import (BandScaling, DecayAttentionSpec, DualScanSpec, OutputNormBlockSpec,
-                    ParallelMixerSpec, PostNormBlockSpec, QueryTemperature, SelectiveScanSpec,
+from .specs import (BandScaling, BigramSpec, DecayAttentionSpec, DualScanSpec, GatedDeltaSpec,
+                    OutputNormBlockSpec, ParallelBlockSpec, ParallelMixerSpec, PostNormBlockSpec, QueryTemperature, SelectiveScanSpec,
                     WindowSinkAttentionSpec)
 from .specs import (AttentionSpec, BlockSpec, ClampedExpertSpec, ConfigError, DeltaRuleSpec,
                     DenseMLPSpec, DifferentialAttentionSpec, GatedMLPSpec, LatentAttentionSpec,
@@ -15,6 +15,7 @@ from .venanex import VenanexConfig
 from .zodirax import ZodiraxConfig
 from .gesuvik import GesuvikConfig
 from .felovik import FelovikConfig
+from .gozolix import GozolixConfig
 
 __all__ = ["AttentionSpec", "BlockSpec", "ConfigError", "DeltaRuleSpec", "DenseMLPSpec",
            "GatedMLPSpec", "LayerCall", "LogDistanceAttentionSpec", "ModelSpec", "NormSpec",
@@ -22,6 +23,7 @@ __all__ = ["AttentionSpec", "BlockSpec", "ConfigError", "DeltaRuleSpec", "DenseM
            "LatentAttentionSpec", "RampScaling", "RoutedExpertsSpec", "SandwichBlockSpec",
            "BandScaling", "DecayAttentionSpec", "OutputNormBlockSpec", "ParallelMixerSpec",
            "SelectiveScanSpec", "WindowSinkAttentionSpec", "DualScanSpec", "PostNormBlockSpec",
-           "QueryTemperature", "FelovikConfig", "ZodiraxConfig", "GesuvikConfig",
+           "QueryTemperature", "BigramSpec", "GatedDeltaSpec", "ParallelBlockSpec", "GozolixConfig",
+           "FelovikConfig", "ZodiraxConfig", "GesuvikConfig",
            "Qwen2Config", "TebonexConfig", "VenanexConfig", "architecture_name", "config_from_dict",
            "config_from_folder", "known_architectures", "register_architecture"]

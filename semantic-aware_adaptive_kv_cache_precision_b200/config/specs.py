@@ -244,8 +244,9 @@ class RoutedExpertsSpec:
     without it. `identity` n: the router has n more outputs after the experts'; an "expert"
     chosen among them has no tensors and returns its input (times the weight).
     `groups` g: the router's outputs form g equal groups of neighbours, a group's score is the
-    largest in it, and only the outputs of the `keep_groups` best groups can be chosen.
-    `renormalize`: the chosen scores are divided by (their sum + 1e-20). `weight_input`: the
+    sum of the `group_top` (1 or 2) largest in it, and only the outputs of the `keep_groups` best
+    groups can be chosen. `renormalize`: the chosen scores are divided by (their sum + 1e-20).
+    `scale` multiplies the weights. `weight_input`: the
     score multiplies the expert's input (out = sum expert(w x)) rather than its output.
     `shared`: one more expert that every token uses, multiplied by `sigmoid(Wsg x)`, one
     number a token (`shared.sg`), if `shared_gate`.
@@ -265,6 +266,8 @@ class RoutedExpertsSpec:
     identity: int = 0
     groups: int = 1
     keep_groups: int = 1
+    group_top: int = 1
+    scale: float = 1.0
     kind: str = "routed_experts"
 
 
@@ -285,7 +288,8 @@ class WindowSinkAttentionSpec:
         weights_ij = exp(s_ij) / (sum_visible exp(s_ij') + exp(sink[h])),   s_ij = q_i . k_j * scale
 
     (`window` None: every earlier key; `sink` False: the plain softmax). Kept tokens keep their
-    true positions. `qk_norm` "whole": queries and keys are each divided by the root mean square
+    true positions. `softcap` c: the score becomes `c tanh(s / c)`; `slopes` (one number a head):
+    then `slopes[h] * (i - j)` is taken off it. `qk_norm` "whole": queries and keys are each divided by the root mean square
     of their WHOLE projection (all heads together, `eps` inside the root) and multiplied by a
     weight of that size, before the rotation; "head": each head by its own root mean square,
     without a weight; None: no norm. `q_temp`: queries are multiplied by a number of their
@@ -293,7 +297,8 @@ class WindowSinkAttentionSpec:
     read from the mixer's input, before the output projection. `position`: a rotation of the first
     `rotary_dim` numbers of every head, or None. Values may have a width of their own; `bias`:
     q, k, v have biases. The heads' outputs are multiplied by `out_scale` before the output
-    projection.
+    projection. `own_kv` False: the layer has no projections of keys and values; its layer call
+    names the cache entry of another attention layer with the same key/value heads and widths.
 
     Tensor names after the part's prefix: `q`, `k`, `v` (+ `.b`), `g`, `q.norm`, `k.norm`,
     `sink`, `o`."""
@@ -313,6 +318,9 @@ class WindowSinkAttentionSpec:
     out_scale: float = 1.0
     q_temp: Optional[QueryTemperature] = None
     gate: bool = False
+    softcap: Optional[float] = None
+    slopes: Optional[tuple] = None
+    own_kv: bool = True
     kind: str = "window_sink_attention"
 
 
@@ -421,8 +429,38 @@ class DualScanSpec:
 
 
 @dataclass(frozen=True)
+class GatedDeltaSpec:
+    """The gated delta rule (a linear recurrence whose state is a matrix a head): q and k
+    (`kv_heads x head_dim`) and v (`heads x value_dim`) each pass a causal convolution a channel
+    over `taps` tokens (last column: the current token; zeros before the start) and silu; q and k
+    become unit vectors a head, x / sqrt(sum(x^2) + `unit_eps`), and q is multiplied by `q_scale`;
+    `g = exp(-exp(A_log) softplus(Wa h + dt_bias))` and `beta = sigmoid(Wb h)`, one number a head;
+    per head, which reads q and k of head floor(h / (heads / kv_heads)),
+
+        S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+
+    Each head's o is divided by its root mean square (`eps` inside the root), multiplied by a
+    weight of `value_dim` numbers that the heads share and by `silu(Wg h)`, and projected. State a
+    sequence: S (fp32) and the convolutions' last `taps - 1` inputs.
+
+    Tensor names after the part's prefix: `q`, `k`, `v` (+ `.conv`), `g`, `a`, `b`, `A_log`,
+    `dt_bias`, `norm`, `o`."""
+    hidden: int
+    heads: int
+    kv_heads: int
+    head_dim: int
+    value_dim: int
+    taps: int
+    q_scale: float
+    eps: float
+    unit_eps: float = 1e-6
+    kind: str = "gated_delta"
+
+
+@dataclass(frozen=True)
 class DenseMLPSpec:
-    """Dense feed-forward without a gate: `down(act(up(x)))`; tensors `up` and `down`."""
+    """Dense feed-forward without a gate: `down(act(up(x)))`; tensors `up` and `down`.
+    `activation` "gelu_tanh" or "relu_squared"."""
     hidden: int
     intermediate: int
     activation: str = "gelu_tanh"
@@ -447,6 +485,23 @@ class BlockSpec:
     mixer_norm_name: str = "input_layernorm"
     ffn_norm_name: str = "post_attention_layernorm"
     kind: str = "pre_norm"
+
+
+@dataclass(frozen=True)
+class ParallelBlockSpec:
+    """A layer whose two sublayers read the output of ONE norm and are added together:
+
+        h = norm(x);   x += mixer(h) + ffn(h)
+
+    `ffn` None: the layer has no feed-forward."""
+    prefix: str
+    mixer: object
+    ffn: object
+    norm: NormSpec
+    mixer_name: str = "mix"
+    ffn_name: str = "mlp"
+    norm_name: str = "norm1"
+    kind: str = "parallel_block"
 
 
 @dataclass(frozen=True)
@@ -553,6 +608,18 @@ class LayerCall:
 
 
 @dataclass(frozen=True)
+class BigramSpec:
+    """A second embedding, of pairs of tokens: the table `name` ([buckets + 1, hidden]) adds its
+    row `(previous token * mul_prev + token * mul_cur) mod buckets` to a token's (scaled)
+    embedding row, and its last row to a sequence's first token. The previous token is part of a
+    sequence's state in the cache."""
+    name: str
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass(frozen=True)
 class ModelSpec:
     """`embed_scale` multiplies the embedding's rows as they enter the residual stream;
     `logit_scale` multiplies the logits and `logit_softcap` c then bends them to
@@ -561,7 +628,8 @@ class ModelSpec:
     of this architecture may hold without any part reading them (buffers that exporters
     write, such as a rotary table's `inv_freq`); anything else unexpected is an error.
     `position_name` names a table [max_positions, hidden] of learned position vectors that are
-    added to the (scaled) embedding rows; None: there is none."""
+    added to the (scaled) embedding rows; None: there is none. `bigram`: a table of pairs of
+    tokens that is added to them as well."""
     architecture: str
     vocab_size: int
     hidden: int
@@ -584,6 +652,7 @@ class ModelSpec:
     streams: int = 1
     input_mix_name: Optional[str] = None
     position_name: Optional[str] = None
+    bigram: Optional[BigramSpec] = None
 
     def cache_entries(self) -> int:
         return 1 + max((c.cache for c in self.run_order), default=-1)

@@ -23,7 +23,8 @@
 //   * several softmax maps a head over the same values (MAPS = 2: the key row holds one key
 //     a map, queries lie head by head as [map 1 | map 2]) combined as
 //       o = a1 - lambda * a2;  out = o / sqrt(mean(o^2) + eps) * out_scale * sigmoid(gate)
-//     with the gate taken element by element from the projection's output.
+//     with the gate taken element by element from the projection's output;
+//   * a soft cap on the scores, and a penalty that grows linearly with the distance.
 #include "common.cuh"
 
 // What the tiled kernel needs beyond the plain grouped-query case; `attention_extra_plain`
@@ -69,6 +70,10 @@ struct AttentionExtra {
   // h's output is multiplied by sigmoid(elem_gate[t * stride + h * vdim + c]). Null: none.
   const float* elem_gate;
   long long elem_gate_stride;
+  // softcap c > 0: a score s becomes c tanh(s / c). linear (fp32, one number a head; null: none):
+  // then linear[h] * (i - j) is taken off it.
+  float softcap;
+  const float* linear;
 };
 
 namespace {
@@ -236,6 +241,14 @@ __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, flo
   }
 }
 
+// cap * tanh(s / cap). 32-bit keys: the library's tanhf; 16-bit keys: 1 - 2 / (e^(2z) + 1), whose
+// error (some 2e-7 of the cap) is far below what the rounded keys leave in the score.
+template <typename T>
+__device__ __forceinline__ float soft_cap(float s, float cap) {
+  if (sizeof(T) == 4) return cap * tanhf(s / cap);
+  return cap * (1.f - __fdividef(2.f, __expf(2.f * __fdividef(s, cap)) + 1.f));
+}
+
 template <int P, int VPL, int MAPS, typename T>
 __global__ void __launch_bounds__(VPL >= 16 ? 256 : 512)      // (wide values: more registers)
 distance_attention_tiled_kernel(
@@ -314,6 +327,8 @@ distance_attention_tiled_kernel(
       if (p < np && slope) {
         sl[p] = slope[h0 + p];
         rt[p] = rate[h0 + p];
+      } else if (p < np && x.linear) {
+        sl[p] = x.linear[(h0 + p) / MAPS];
       }
       const T* qa = qkv + (long long)t * stride + (long long)(h0 + p) * x.q_head_stride;
       const T* qb = q2 ? q2 + (long long)t * x.q2_stride +
@@ -376,7 +391,9 @@ distance_attention_tiled_kernel(
         float sc = -INFINITY;
         if (valid) {
           sc = s[p] * scale;
+          if (x.softcap > 0.f) sc = soft_cap<T>(sc, x.softcap);
           if (slope) sc -= sl[p] * log1pf(rt[p] * dist);
+          else if (x.linear) sc = fmaf(-sl[p], dist, sc);
         }
         const float m_new = fmaxf(m[p], warp_max(sc));
         const float corr = expf(m[p] - m_new);
@@ -880,7 +897,8 @@ SAKV_EXPORT int sakv_distance_attention(const void* qkv, int dtype, long long st
 // token, kv head and group of heads; zero on entry, left zero) tells which block came last.
 // `heads_first` (with splits 1): the form for decoded tokens in which a block's warps are one
 // token's groups of heads and share each chunk of keys through shared memory; `key_splits`
-// blocks then take contiguous shares of the chunks.
+// blocks then take contiguous shares of the chunks. softcap (0: none) and linear (fp32 [heads] or
+// null) as in `AttentionExtra`.
 SAKV_EXPORT int sakv_cached_attention(
     const void* qkv, int dtype, long long stride, int q_head_stride, const void* q2,
     long long q2_stride, int q2_head_stride, int q_split, int gate_off, void* out,
@@ -890,8 +908,9 @@ SAKV_EXPORT int sakv_cached_attention(
     int window, int chunk, float lambda, float out_scale, float eps, int gate_elem_off,
     int splits, int key_splits, float* scratch, long long scratch_floats, int* tickets,
     int warp_stage, int heads_first, int keep_first, const float* sink, const void* head_gate,
-    long long head_gate_stride, const float* elem_gate, long long elem_gate_stride,
-    cudaStream_t stream) {
+    long long head_gate_stride, const float* elem_gate, long long elem_gate_stride, float softcap,
+    const float* linear, cudaStream_t stream) {
+  if (softcap < 0.f) return cudaErrorInvalidValue;
   if (elem_gate != nullptr && maps != 1) return cudaErrorInvalidValue;
   if (keep_first < 0 || (keep_first > 0 && chunk > 0)) return cudaErrorInvalidValue;
   if (head_gate != nullptr && (maps != 1 || gate_off >= 0)) return cudaErrorInvalidValue;
@@ -930,6 +949,8 @@ SAKV_EXPORT int sakv_cached_attention(
   x.head_gate_stride = head_gate_stride;
   x.elem_gate = elem_gate;
   x.elem_gate_stride = elem_gate_stride;
+  x.softcap = softcap;
+  x.linear = linear;
   const void* values = x.v_in_k ? k_cache : v_cache;
   if (dtype == SAKV_F32)
     return pick_tiled<float>(qkv, stride, gate_off, out, k_cache, values, positions, token_seq,

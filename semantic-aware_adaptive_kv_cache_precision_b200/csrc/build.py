@@ -56,6 +56,7 @@ LIBRARIES = {
     "norm_update": "norm_update.cu",
     "qk_prepare": "qk_prepare.cu",
     "recurrent_scan": "recurrent_scan.cu",
+    "gated_delta": "gated_delta.cu",
 }
 
 #: extra flags of single libraries (libraries that need the driver API, for instance)

@@ -30,6 +30,42 @@ __global__ void embed_kernel(const int32_t* __restrict__ ids, const Table* __res
   }
 }
 
+// The embedding with a second table of pairs of tokens: out[t] = table[ids[t]] * scale +
+// pairs[(previous * mul_prev + ids[t] * mul_cur) mod buckets], a sequence's first token taking the
+// pairs' last row (number `buckets`). The token before a sequence's part in this step is kept in
+// `last` (one number a slot); the block of the part's first token reads it and then leaves the
+// part's last token there, so nobody else touches it. One block a token.
+template <typename Table>
+__global__ void embed_pairs_kernel(const int32_t* __restrict__ ids, const Table* __restrict__ table,
+                                   float* __restrict__ out, int hidden, int vocab, float scale,
+                                   const Table* __restrict__ pairs, long long buckets,
+                                   long long mul_prev, long long mul_cur,
+                                   const int32_t* __restrict__ positions,
+                                   const int32_t* __restrict__ token_seq,
+                                   const int32_t* __restrict__ cu_seqlens,
+                                   const int32_t* __restrict__ slots, int32_t* __restrict__ last) {
+  __shared__ long long shared_row;
+  let_next_kernel_start();
+  wait_for_previous_kernel();
+  const long long t = blockIdx.x;
+  const int id = ids[t];
+  if (threadIdx.x == 0) {
+    const int b = token_seq[t];
+    const bool starts = t == cu_seqlens[b];            // the first of its part
+    long long previous = starts ? last[slots[b]] : ids[t - 1];
+    if (starts) last[slots[b]] = ids[cu_seqlens[b + 1] - 1];
+    long long row = (previous * mul_prev + id * mul_cur) % buckets;
+    if (row < 0) row += buckets;
+    shared_row = positions[t] == 0 ? buckets : row;
+  }
+  __syncthreads();
+  const Table* pair = pairs + shared_row * hidden;
+  const Table* own = table + (long long)id * hidden;
+  const bool known = id >= 0 && id < vocab;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x)
+    out[t * hidden + c] = (known ? widen(own[c]) * scale : 0.f) + widen(pair[c]);
+}
+
 // gate_up[t, 0:I] = gate, gate_up[t, I:2I] = up  ->  out[t, 0:I]
 template <typename T>
 __global__ void gated_silu_kernel(const T* __restrict__ gate_up, T* __restrict__ out,
@@ -129,7 +165,75 @@ __global__ void gelu_tanh_kernel(const T* __restrict__ in, T* __restrict__ out, 
   }
 }
 
+// relu(z)^2, the same way.
+template <typename T>
+__global__ void relu_squared_kernel(const T* __restrict__ in, T* __restrict__ out,
+                                    long long count) {
+  let_next_kernel_start();
+  wait_for_previous_kernel();
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < count;
+       i += (long long)gridDim.x * blockDim.x) {
+    const float z = fmaxf(widen(in[i]), 0.f);
+    out[i] = narrow<T>(z * z);
+  }
+}
+
+__global__ void relu_squared_bf16x8_kernel(const uint4* __restrict__ in, uint4* __restrict__ out,
+                                           long long count8) {
+  let_next_kernel_start();
+  wait_for_previous_kernel();
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < count8;
+       i += (long long)gridDim.x * blockDim.x) {
+    uint4 v = in[i];
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      float2 f = __bfloat1622float2(h[j]);
+      f.x = fmaxf(f.x, 0.f);
+      f.y = fmaxf(f.y, 0.f);
+      h[j] = __floats2bfloat162_rn(f.x * f.x, f.y * f.y);
+    }
+    out[i] = v;
+  }
+}
+
 }  // namespace
+
+// out = relu(in)^2 (in place is fine).
+SAKV_EXPORT int sakv_relu_squared(const void* in, void* out, int dtype, long long count,
+                                  cudaStream_t stream) {
+  if (count < 0) return cudaErrorInvalidValue;
+  if (count == 0) return 0;
+  if (dtype == SAKV_BF16 && count % 8 == 0 && !(((uintptr_t)in | (uintptr_t)out) & 15))
+    return launch_overlapped(relu_squared_bf16x8_kernel, dim3(grid_for(count / 8, 256)), dim3(256),
+                             0, stream, 1, (const uint4*)in, (uint4*)out, count / 8);
+  const dim3 grid(grid_for(count, 256)), block(256);
+  if (dtype == SAKV_F32)
+    return launch_overlapped(relu_squared_kernel<float>, grid, block, 0, stream, 1,
+                             (const float*)in, (float*)out, count);
+  if (dtype == SAKV_BF16)
+    return launch_overlapped(relu_squared_kernel<__nv_bfloat16>, grid, block, 0, stream, 1,
+                             (const __nv_bfloat16*)in, (__nv_bfloat16*)out, count);
+  return cudaErrorInvalidValue;
+}
+
+// pairs: [buckets + 1, hidden] of the table's type; last: int32 [slots], the token each sequence
+// brought last, read and replaced.
+SAKV_EXPORT int sakv_embed_pairs(const int32_t* ids, const void* table, int table_dtype, float* out,
+                                 int tokens, int hidden, int vocab, float scale, const void* pairs,
+                                 long long buckets, long long mul_prev, long long mul_cur,
+                                 const int32_t* positions, const int32_t* token_seq,
+                                 const int32_t* cu_seqlens, const int32_t* slots, int32_t* last,
+                                 cudaStream_t stream) {
+  if (tokens < 0 || hidden <= 0 || vocab <= 0 || buckets <= 0) return cudaErrorInvalidValue;
+  if (tokens == 0) return 0;
+  const dim3 grid(tokens), block(hidden >= 1024 ? 256 : 128);
+#define SAKV_PAIRS(T)                                                                              return launch_overlapped(embed_pairs_kernel<T>, grid, block, 0, stream, 1, ids, (const T*)table,                            out, hidden, vocab, scale, (const T*)pairs, buckets, mul_prev, mul_cur,                            positions, token_seq, cu_seqlens, slots, last)
+  if (table_dtype == SAKV_F32) SAKV_PAIRS(float);
+  if (table_dtype == SAKV_BF16) SAKV_PAIRS(__nv_bfloat16);
+#undef SAKV_PAIRS
+  return cudaErrorInvalidValue;
+}
 
 SAKV_EXPORT int sakv_gelu_tanh(const void* in, void* out, int dtype, long long count,
                                cudaStream_t stream) {

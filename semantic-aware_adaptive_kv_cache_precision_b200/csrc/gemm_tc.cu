@@ -17,6 +17,7 @@
 //                                                      matrix, two accumulators side by side
 //   gated_clamped      : g sigmoid(alpha g) (u + plus) with g = min(C_gate, limit), u = C_up
 //                        within +-limit
+//   relu_squared       : max(C + bias, 0)^2            the up rows of a feed-forward without gate
 //
 // With few tokens and a small N there are too few row tiles to fill the GPU's SMs, so K is
 // split over the blocks of a thread-block cluster (up to 8, along blockIdx.z): every
@@ -40,7 +41,7 @@ constexpr int kThreads = 224;      // warps: 0 TMA, 1 and 6 MMA issue, 2..5 epil
 constexpr int kWTile = BM * BK * 2;
 constexpr int kMaxSplits = 8;     // portable cluster size
 
-enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_ACCUM = 2, EPI_GATED = 3, EPI_CLAMPED = 4 };
+enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_ACCUM = 2, EPI_GATED = 3, EPI_CLAMPED = 4, EPI_RELU2 = 5 };
 constexpr bool gated_epi(int epi) { return epi == EPI_GATED || epi == EPI_CLAMPED; }
 
 struct Params {
@@ -130,6 +131,9 @@ __device__ __forceinline__ void finish(const Params& p, int part, int m, int n, 
     atomicAdd(reinterpret_cast<float*>(p.out) + at, c + bias);
   } else if (kEpi == EPI_CLAMPED) {
     reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(clamped(p, c, up));
+  } else if (kEpi == EPI_RELU2) {
+    const float z = fmaxf(c + bias, 0.f);
+    reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(z * z);
   } else {
     const float silu = c / (1.0f + expf(-c));
     reinterpret_cast<__nv_bfloat16*>(p.out)[at] = __float2bfloat16_rn(silu * up);
@@ -216,6 +220,9 @@ __device__ __forceinline__ void finish4(const Params& p, int part, int m, int n,
       const float g[4] = {c.x, c.y, c.z, c.w}, u[4] = {up.x, up.y, up.z, up.w};
 #pragma unroll
       for (int i = 0; i < 4; ++i) r[i] = clamped(p, g[i], u[i]);
+    } else if (kEpi == EPI_RELU2) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) r[i] = fmaxf(r[i], 0.f) * fmaxf(r[i], 0.f);
     }
     *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.out) + at) =
         make_uint2(mma::pack_bf16(r[0], r[1]), mma::pack_bf16(r[2], r[3]));
@@ -539,7 +546,7 @@ SAKV_EXPORT int sakv_gemm_tc(const void* w_map, const void* x_map, int M, int N,
                              int splits, int parts, int epi, int dual_offset, const void* bias,
                              int bias_dtype, void* out, long long ldo, long long part_stride,
                              float limit, float alpha, float plus, cudaStream_t stream) {
-  if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || splits < 1 || epi < 0 || epi > EPI_CLAMPED ||
+  if (M <= 0 || N <= 0 || K <= 0 || (K % 8) || splits < 1 || epi < 0 || epi > EPI_RELU2 ||
       ldo < N || parts < 1 || parts > 64 || (parts > 1 && epi != EPI_F32))
     return cudaErrorInvalidValue;
   const int total_kb = (K + BK - 1) / BK;
@@ -572,6 +579,7 @@ SAKV_EXPORT int sakv_gemm_tc(const void* w_map, const void* x_map, int M, int N,
   if (mt == MT_)                                                                  \
     return epi == EPI_CLAMPED ? launch<MT_, EPI_CLAMPED>(wm, xm, p, n_tiles, m_tiles, stream)     \
          : dual ? launch<MT_, EPI_GATED>(wm, xm, p, n_tiles, m_tiles, stream)     \
+         : epi == EPI_RELU2 ? launch<MT_, EPI_RELU2>(wm, xm, p, n_tiles, m_tiles, stream) \
          : epi == EPI_BF16 ? launch<MT_, EPI_BF16>(wm, xm, p, n_tiles, m_tiles, stream)   \
          : epi == EPI_F32 ? launch<MT_, EPI_F32>(wm, xm, p, n_tiles, m_tiles, stream)     \
                           : launch<MT_, EPI_ACCUM>(wm, xm, p, n_tiles, m_tiles, stream)

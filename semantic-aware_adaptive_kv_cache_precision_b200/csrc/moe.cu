@@ -4,8 +4,9 @@
 //            scores as weights, and the token's place among the rows of each chosen expert.
 //            A score is the sigmoid of the logit, or the softmax over all the router's
 //            outputs; a bias an output may be added for the choice only. The outputs may form
-//            groups of neighbours of which only the best few (by their largest score) are open
-//            to a token's choice, and the chosen scores may be divided by their sum. Outputs beyond the
+//            groups of neighbours of which only the best few (by their largest score, or the sum
+//            of their two largest) are open to a token's choice, and the chosen scores may be
+//            divided by their sum and multiplied by a constant. Outputs beyond the
 //            experts that have weights are identity experts: they take no rows, and combine
 //            adds the token's own input times the weight for them
 //   plan     one block: where each expert's rows begin and which (expert, first row) every
@@ -56,13 +57,16 @@ __global__ void logits_kernel(const T* __restrict__ h, const float* __restrict__
 // is sigmoid(z); 1: exp(z - max) / sum over all outputs. bias (null: none): added to the score
 // for the choice. Without a bias the scores' order is the logits' own, and they are compared.
 // groups > 1: the outputs form that many equal groups of neighbours; the `keep` groups with the
-// largest best score (of the choice) are open, the rest closed (ties: the lowest index).
-// renorm: the weights are the chosen scores over (their sum + 1e-20).
+// largest best score (of the choice; with `group_top` 2 the largest sum of their two best) are
+// open, the rest closed (ties: the lowest index). renorm: the weights are the chosen scores over
+// (their sum + 1e-20). scale multiplies the weights.
 struct RouteForm {
   int softmax;
   const float* bias;
   int groups, keep;            // groups <= 64
   int renorm;
+  int group_top;               // 1 or 2
+  float scale;
 };
 
 __device__ __forceinline__ void route_token(const float* __restrict__ z, int experts, int top,
@@ -95,7 +99,17 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int exp
       for (int g = lane; g < form.groups; g += 32) {
         if (open >> g & 1) continue;
         float v = -INFINITY;
-        for (int e = g * per_group; e < (g + 1) * per_group; ++e) v = fmaxf(v, rank_of(e));
+        if (form.group_top == 2) {                   // (sums are of scores, never of logits)
+          float second = -INFINITY;
+          for (int e = g * per_group; e < (g + 1) * per_group; ++e) {
+            const float r = by_logit ? score(z[e]) : rank_of(e);
+            second = fmaxf(second, fminf(v, r));
+            v = fmaxf(v, r);
+          }
+          if (per_group > 1) v += second;
+        } else {
+          for (int e = g * per_group; e < (g + 1) * per_group; ++e) v = fmaxf(v, rank_of(e));
+        }
         if (v > best || at == 0x7fffffff) {
           best = v;
           at = g;
@@ -145,8 +159,10 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int exp
       rank[k] = at < real ? atomicAdd(counts + at, 1) : -1;
     }
   }
-  if (form.renorm && lane == 0)
-    for (int k = 0; k < top; ++k) weights[k] /= sum_chosen + 1e-20f;
+  if ((form.renorm || form.scale != 1.f) && lane == 0) {
+    const float by = form.renorm ? sum_chosen + 1e-20f : 1.f;
+    for (int k = 0; k < top; ++k) weights[k] = weights[k] / by * form.scale;
+  }
 }
 
 __global__ void route_kernel(const float* __restrict__ logits, long long ld, int experts, int top,
@@ -464,8 +480,8 @@ __global__ void combine_kernel(const float* __restrict__ rows, const int32_t* __
 
 SAKV_EXPORT int sakv_moe_tile_rows() { return TM; }
 
-static bool form_fits(int experts, int top, int groups, int keep) {
-  return groups >= 1 && groups <= 64 && experts % groups == 0 && keep >= 1 && keep <= groups &&
+static bool form_fits(int experts, int top, int groups, int keep, int group_top) {
+  return (group_top == 1 || group_top == 2) && groups >= 1 && groups <= 64 && experts % groups == 0 && keep >= 1 && keep <= groups &&
          (long long)experts / groups * keep >= top;
 }
 
@@ -473,20 +489,21 @@ static bool form_fits(int experts, int top, int groups, int keep) {
 // experts with weights and the rest to identity experts); counts: int32 [real], zero on entry
 // (plan leaves it zero again). chosen, rank: int32 [tokens, top] (rank -1: an identity
 // expert); weights: fp32. softmax: the score's kind; bias: fp32 [experts] or null; groups, keep,
-// renorm: see `RouteForm`.
+// renorm, group_top, scale: see `RouteForm`.
 SAKV_EXPORT int sakv_moe_route(const float* logits, long long ld, int experts, int top,
                                int32_t* chosen, float* weights, int32_t* counts, int32_t* rank,
                                int tokens, int real, int softmax, const float* bias, int groups,
-                               int keep, int renorm, cudaStream_t stream) {
+                               int keep, int renorm, int group_top, float scale,
+                               cudaStream_t stream) {
   if (tokens < 0 || experts <= 0 || experts > 1024 || top <= 0 || top > experts || top > 32 ||
-      ld < experts || real < 0 || real > experts || !form_fits(experts, top, groups, keep))
+      ld < experts || real < 0 || real > experts || !form_fits(experts, top, groups, keep, group_top))
     return cudaErrorInvalidValue;
   if (tokens == 0) return 0;
   const int threads = 128;
   const long long blocks = ((long long)tokens * 32 + threads - 1) / threads;
   return launch_ordered(route_kernel, dim3((unsigned)blocks), dim3(threads), 0, stream, logits, ld,
                         experts, top, chosen, weights, counts, rank, tokens, real,
-                        RouteForm{softmax, bias, groups, keep, renorm});
+                        RouteForm{softmax, bias, groups, keep, renorm, group_top, scale});
 }
 
 // `sakv_moe_route` and `sakv_moe_plan` in one launch of one block, for steps of few tokens
@@ -494,16 +511,18 @@ SAKV_EXPORT int sakv_moe_route(const float* logits, long long ld, int experts, i
 SAKV_EXPORT int sakv_moe_route_plan(const float* logits, long long ld, int experts, int top,
                                     int32_t* chosen, float* weights, int32_t* rank, int tokens,
                                     int real, int softmax, const float* bias, int groups,
-                                    int keep, int renorm, int32_t* offsets,
+                                    int keep, int renorm, int group_top, float scale,
+                                    int32_t* offsets,
                                     int32_t* tile_expert, int32_t* tile_row, int32_t* n_tiles,
                                     int max_tiles, cudaStream_t stream) {
   if (tokens <= 0 || experts <= 0 || experts > 1024 || top <= 0 || top > experts || top > 32 ||
       ld < experts || real <= 0 || real > experts || max_tiles <= 0 ||
-      !form_fits(experts, top, groups, keep))
+      !form_fits(experts, top, groups, keep, group_top))
     return cudaErrorInvalidValue;
   return launch_ordered(route_plan_kernel, dim3(1), dim3(256), (size_t)(2 * real + 1) * 4, stream,
                         logits, ld, experts, top, chosen, weights, rank, tokens, real,
-                        RouteForm{softmax, bias, groups, keep, renorm}, offsets, tile_expert, tile_row, n_tiles, max_tiles);
+                        RouteForm{softmax, bias, groups, keep, renorm, group_top, scale}, offsets,
+                        tile_expert, tile_row, n_tiles, max_tiles);
 }
 
 // out[t, o] = sum_i h[t, i] w[o, i] in fp32: h [tokens, width] of `dtype`, w fp32 [outputs,

@@ -9,6 +9,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
+from ..cache.needs import StateNeed
 from ..parts import build_part
 from ..weights import TensorDecl, load_checkpoint, random_arena
 
@@ -29,6 +30,8 @@ class DecoderModel:
             owners.setdefault(call.cache, call.block)
         if sorted(owners) != list(range(len(owners))):
             raise ValueError("cache entries of the run order must be numbered 0, 1, 2, ...")
+        if spec.bigram and spec.position_name:
+            raise ValueError("a table of pairs beside learned positions is not built")
         self._owners = owners
         self.arena = None
         #: whether every part says its step can be captured in a CUDA graph
@@ -41,6 +44,8 @@ class DecoderModel:
         decls = [TensorDecl(spec.embed_name, (spec.vocab_size, spec.hidden))]
         if spec.position_name:
             decls.append(TensorDecl(spec.position_name, (spec.max_positions, spec.hidden)))
+        if spec.bigram:
+            decls.append(TensorDecl(spec.bigram.name, (spec.bigram.buckets + 1, spec.hidden)))
         for block in self.blocks:
             decls += block.tensor_decls()
         decls += self.final_norm.tensor_decls()
@@ -70,6 +75,7 @@ class DecoderModel:
         self.head = self.embed if self.spec.tie_head else arena.view(self.spec.head_name)
         self.head_bias = arena.view(self.spec.head_bias_name) if self.spec.head_bias_name else None
         self.positions = arena.view(self.spec.position_name) if self.spec.position_name else None
+        self.pairs = arena.view(self.spec.bigram.name) if self.spec.bigram else None
         self.input_mix = arena.view(self.spec.input_mix_name) if self.spec.input_mix_name else None
         for block in self.blocks:
             block.bind(arena)
@@ -90,8 +96,10 @@ class DecoderModel:
     # -- cache ------------------------------------------------------------------
 
     def cache_needs(self) -> list:
-        """What each cache entry must hold: the need of the block that owns it."""
-        return [self.blocks[self._owners[e]].cache_need() for e in range(len(self._owners))]
+        """What each cache entry must hold: the need of the block that owns it; behind the blocks'
+        entries, where the embedding reads pairs of tokens, the token a sequence brought last."""
+        needs = [self.blocks[self._owners[e]].cache_need() for e in range(len(self._owners))]
+        return needs + ([StateNeed((1,), "int32")] if self.spec.bigram else [])
 
     def prepare(self, max_positions: int) -> None:
         for block in self.blocks:
@@ -113,10 +121,10 @@ class DecoderModel:
         if streams > 1:          # every stream starts as the embedding's output
             x = torch.empty((streams, step.tokens, self.spec.hidden), dtype=torch.float32,
                             device=self.device)
-            self._embed(step, x[0])
+            self._embed(step, cache, x[0])
             ops.streams_spread(x)
         else:
-            x = self._embed(step)
+            x = self._embed(step, cache)
 
         def stream(x):           # what the streams stand for: their sum
             return ops.streams_step(x, reduce=True) if x.dim() == 3 else x.clone()
@@ -159,9 +167,15 @@ class DecoderModel:
             _settle(x, pending)
         return ops.streams_step(x, reduce=True) if x.dim() == 3 else x
 
-    def _embed(self, step, out=None) -> torch.Tensor:
+    def _embed(self, step, cache, out=None) -> torch.Tensor:
         """The stream at the start: the tokens' rows of the embedding times its scale, plus
-        the learned vectors of their positions where the model has them."""
+        the learned vectors of their positions, or the rows of a table of pairs of tokens, where
+        the model has them."""
+        if self.pairs is not None:
+            last = cache.entry_view(len(self._owners), step.tables).state
+            b = self.spec.bigram
+            return ops.embed_pairs(step, self.embed, self.pairs, b.mul_prev, b.mul_cur, last,
+                                   out=out, scale=self.spec.embed_scale)
         if self.positions is not None and step.max_position >= self.positions.shape[0]:
             raise ValueError(f"position {step.max_position} is beyond the model's "
                              f"{self.positions.shape[0]} learned positions")

@@ -12,10 +12,10 @@ import torch
 
 from ._lib import (BF16, CACHE_BLOCK, F32, KernelError, call, dtype_code, plain_function, ptr,
                    require_cuda)
-from .linear import Deferred, gated_up, linear, per_head
+from .linear import Deferred, dense_up, gated_up, linear, per_head
 from . import gemm_tc
 from .streams import streams_spread, streams_step, token_shift
-from .recurrent import delta_rule
+from .recurrent import delta_rule, gated_delta
 from .scan import causal_conv, decay_attention, dual_scan, norm_gate, selective_scan, step_size
 from . import mixture
 from .mixture import latent_prepare, rotate_heads
@@ -28,7 +28,7 @@ __all__ = ["CACHE_BLOCK", "KernelError", "embed", "rms_norm", "rope_store", "att
            "attention_decode", "attention_prefill", "attention_prefill_tc", "tc_prefill_takes", "plan_wide_tiles", "upload_wide_plan",
            "upload_query_tiles",
            "decode_splits", "plan_token_blocks", "fast_path_takes", "forget_descriptors",
-           "kernel_errors", "gated_silu", "gelu_tanh", "streams_step", "streams_spread", "token_shift",
+           "kernel_errors", "gated_silu", "gelu_tanh", "relu_squared", "dense_up", "embed_pairs", "gated_delta", "streams_step", "streams_spread", "token_shift",
            "delta_rule", "kv_store", "layer_norm", "cached_attention", "mixture", "latent_prepare",
            "rotate_heads", "distance_attention", "rms_update", "rms_join", "qk_prepare", "causal_conv",
            "decay_attention", "dual_scan", "norm_gate", "selective_scan", "step_size", "gated_up", "gemm_tc", "add_into", "scale_cap_", "linear", "per_head", "choose", "Deferred"]
@@ -64,6 +64,33 @@ def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None = Non
          hidden, vocab, float(scale), ptr(position_table),
          ptr(positions) if position_table is not None else None,
          0 if position_table is None else position_table.shape[0])
+    return out
+
+
+def embed_pairs(step, table: torch.Tensor, pairs: torch.Tensor, mul_prev: int, mul_cur: int,
+                last: torch.Tensor, out: torch.Tensor | None = None,
+                scale: float = 1.0) -> torch.Tensor:
+    """The embedding of a step's tokens with a second table of pairs of tokens (`pairs` [buckets
+    + 1, hidden] of the table's type): fp32 `table[id] * scale + pairs[(previous * mul_prev + id *
+    mul_cur) mod buckets]`, a sequence's first token taking the last row of `pairs`. `last` (int32
+    [slots, 1]): the token each sequence brought last, read and replaced."""
+    require_cuda(step.token_ids, table, pairs, last)
+    _check(table.dim() == 2 and table.is_contiguous(), "table: contiguous [vocab, hidden]")
+    vocab, hidden = table.shape
+    tokens = step.token_ids.numel()
+    _check(pairs.dim() == 2 and pairs.is_contiguous() and pairs.shape[1] == hidden
+           and pairs.shape[0] > 1 and pairs.dtype == table.dtype,
+           "pairs: contiguous [buckets + 1, hidden] of the table's type")
+    _check(last.dtype == torch.int32 and last.is_contiguous() and last.numel() == last.shape[0],
+           "last: int32 [slots, 1]")
+    if out is None:
+        out = torch.empty((tokens, hidden), dtype=torch.float32, device=table.device)
+    _check(out.dtype == torch.float32 and out.is_contiguous() and out.shape == (tokens, hidden),
+           "out: fp32 [T, hidden]")
+    call("sakv_embed_pairs", ptr(step.token_ids), ptr(table), dtype_code(table.dtype), ptr(out),
+         tokens, hidden, vocab, float(scale), ptr(pairs), pairs.shape[0] - 1, int(mul_prev),
+         int(mul_cur), ptr(step.positions), ptr(step.token_seq), ptr(step.cu_seqlens),
+         ptr(step.slots), ptr(last))
     return out
 
 
@@ -166,6 +193,16 @@ def gelu_tanh(x: torch.Tensor) -> torch.Tensor:
     _check(x.is_contiguous(), "gelu_tanh: contiguous input")
     out = torch.empty_like(x)
     call("sakv_gelu_tanh", ptr(x), ptr(out), dtype_code(x.dtype), x.numel())
+    return out
+
+
+def relu_squared(x: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+    """`max(x, 0)^2`, element by element (fp32 inside, x's type outside); `out` may be x."""
+    require_cuda(x, out)
+    out = torch.empty_like(x) if out is None else out
+    _check(x.is_contiguous() and out.is_contiguous() and out.shape == x.shape
+           and out.dtype == x.dtype, "relu_squared: contiguous, out like x")
+    call("sakv_relu_squared", ptr(x), ptr(out), dtype_code(x.dtype), x.numel())
     return out
 
 
@@ -337,7 +374,8 @@ def qk_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: in
     rotation), keys and values stored in the cache blocks. Returns the queries [T, heads *
     dim] of `out_dtype`. `norm` "head": every head is divided by its own root mean square
     (`q_weight`, `k_weight`: [dim], the same for all heads, or None: no weight).
-    `temperature` (fp32 [positions]): queries are multiplied by their position's number."""
+    `temperature` (fp32 [positions]): queries are multiplied by their position's number. Without
+    `write_cache` keys and values are not read (`k_off`, `v_off` mean nothing)."""
     require_cuda(proj, q_weight, k_weight, cos, sin, positions, token_seq, block_table, k_cache,
                  v_cache, temperature)
     _check(norm in (None, "whole", "head"), "norm: 'whole', 'head' or None")
@@ -346,8 +384,9 @@ def qk_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: in
     tokens = proj.shape[0]
     _check(proj.dtype == torch.float32 and proj.dim() == 2 and proj.stride(1) == 1,
            "proj: fp32 [T, columns] with contiguous rows")
-    _check(max(q_off + heads * dim, k_off + kv_heads * dim, v_off + kv_heads * vdim)
-           <= proj.shape[1], "queries, keys or values reach beyond proj's columns")
+    _check(q_off + heads * dim <= proj.shape[1]
+           and (not write_cache or max(k_off + kv_heads * dim, v_off + kv_heads * vdim)
+                <= proj.shape[1]), "queries, keys or values reach beyond proj's columns")
     _check((q_weight is None) == (k_weight is None), "q_weight and k_weight come together")
     if q_weight is not None:
         _check(((q_weight.shape == (heads * dim,) and k_weight.shape == (kv_heads * dim,))
@@ -389,7 +428,8 @@ def cached_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      heads_first: bool = False, keep_first: int = 0,
                      sink: torch.Tensor | None = None,
                      head_gate: torch.Tensor | None = None,
-                     elem_gate: torch.Tensor | None = None) -> torch.Tensor:
+                     elem_gate: torch.Tensor | None = None, softcap: float | None = None,
+                     linear_slopes: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of every token of the step over its sequence's cache, in the general
     form of `csrc/attention_distance.cu`: scores, softmax weights and weighted sums in fp32.
 
@@ -415,9 +455,15 @@ def cached_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     shared memory holds them). `heads_first` (with `splits` 1; decode steps): a block's warps
     are ONE token's groups of heads and share every chunk of its keys through shared memory, so
     the rows are read once for all the token's heads; `key_splits` blocks a token then take
-    contiguous shares of the chunks."""
+    contiguous shares of the chunks. `softcap` c: a scaled score s becomes `c tanh(s / c)`;
+    `linear_slopes` (fp32 [heads]): then `slope[h] * (i - j)` is taken off it."""
     require_cuda(q, k_cache, v_cache, positions, token_seq, block_table, q2, sink, head_gate,
-                 elem_gate)
+                 elem_gate, linear_slopes)
+    _check(softcap is None or softcap > 0, "softcap must be positive")
+    _check(linear_slopes is None or (linear_slopes.dtype == torch.float32
+                                     and linear_slopes.shape == (heads,)
+                                     and linear_slopes.is_contiguous()),
+           "linear_slopes: fp32 [heads]")
     tokens = q.shape[0]
     _check(elem_gate is None or (maps == 1 and elem_gate.dtype == torch.float32
                                  and elem_gate.shape == (tokens, heads * vdim)
@@ -474,7 +520,8 @@ def cached_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
          int(splits), int(key_splits), ptr(scratch), floats, ptr(tickets), int(warp_stage),
          int(heads_first), int(keep_first) if window else 0, ptr(sink), ptr(head_gate),
          0 if head_gate is None else head_gate.stride(0), ptr(elem_gate),
-         0 if elem_gate is None else elem_gate.stride(0))
+         0 if elem_gate is None else elem_gate.stride(0), float(softcap or 0.0),
+         ptr(linear_slopes))
     return out
 
 

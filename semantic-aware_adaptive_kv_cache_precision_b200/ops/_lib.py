@@ -26,6 +26,11 @@ SIGNATURES = {
     "sakv_add_into": ("elementwise", [P, P, I, L, P]),
     "sakv_scale_cap": ("elementwise", [P, L, F, F, P]),
     "sakv_gelu_tanh": ("elementwise", [P, P, I, L, P]),
+    "sakv_relu_squared": ("elementwise", [P, P, I, L, P]),
+    "sakv_embed_pairs": ("elementwise", [P, P, I, P, I, I, I, F, P, L, L, L, P, P, P, P, P, P]),
+    "sakv_delta_inputs": ("gated_delta", [P, L, I, I, P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I,
+                                          I, I, F, F, P]),
+    "sakv_delta_scan": ("gated_delta", [P, P, P, P, P, P, P, I, I, I, I, I, I, I, P]),
     "sakv_streams_step": ("streams", [P, L, I, I, I, P, P, P, I, P, P, I, F, P, I, P, P, P, P, I,
                                       P]),
     "sakv_token_shift": ("streams", [P, P, P, I, P, P, P, P, I, I, I, I, P]),
@@ -37,7 +42,8 @@ SIGNATURES = {
                                 [P, I, L, I, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P]),
     "sakv_cached_attention": ("attention_distance",
                               [P, I, L, I, P, L, I, I, I, P, P, I, P, I, P, P, P, I, I, I, I, I, I,
-                               I, F, I, I, F, F, F, I, I, I, P, L, P, I, I, I, P, P, L, P, L, P]),
+                               I, F, I, I, F, F, F, I, I, I, P, L, P, I, I, I, P, P, L, P, L, F, P,
+                               P]),
     "sakv_rms_update": ("norm_update", [P, P, P, F, P, P, F, I, P, I, I, I, F, P]),
     "sakv_rms_join": ("norm_update", [P, P, P, P, P, F, F, F, P, I, F, P, I, I, I, P]),
     "sakv_qk_prepare": ("qk_prepare", [P, L, I, I, I, P, P, I, F, P, P, I, P, P, P, I, P, P, P,
@@ -58,9 +64,10 @@ SIGNATURES = {
                                        I, P]),
     "sakv_rotate_heads": ("latent", [P, I, L, I, I, I, I, P, P, P, I, I, P]),
     "sakv_moe_logits": ("moe", [P, I, P, P, I, I, I, P]),
-    "sakv_moe_route": ("moe", [P, L, I, I, P, P, P, P, I, I, I, P, I, I, I, P]),
+    "sakv_moe_route": ("moe", [P, L, I, I, P, P, P, P, I, I, I, P, I, I, I, I, F, P]),
     "sakv_moe_plan": ("moe", [P, P, P, P, P, I, I, P]),
-    "sakv_moe_route_plan": ("moe", [P, L, I, I, P, P, P, I, I, I, P, I, I, I, P, P, P, P, I, P]),
+    "sakv_moe_route_plan": ("moe", [P, L, I, I, P, P, P, I, I, I, P, I, I, I, I, F, P, P, P, P, I,
+                                    P]),
     "sakv_moe_gather": ("moe", [P, I, P, P, P, P, P, P, I, I, I, I, P]),
     "sakv_moe_product": ("moe", [P, I, P, P, L, P, P, P, P, I, P, I, I, I, F, F, F, P]),
     "sakv_clamped_act": ("moe", [P, P, I, I, I, F, F, F, P]),
@@ -87,6 +94,7 @@ SIGNATURES = {
 PLAIN_SIGNATURES = {
     "sakv_choose_chunks": ("sampling", [I]),
     "sakv_moe_tile_rows": ("moe", []),
+    "sakv_delta_coefficients": ("gated_delta", []),
     "sakv_decode_attention_map": ("attention_decode", [P, P, L, I, I]),
     "sakv_decode_attention_error": ("attention_decode", [P]),
     "sakv_decode_attention_max_cluster": ("attention_decode", [I]),

@@ -9,7 +9,7 @@ import torch
 
 from ._lib import BF16, F32, KernelError, call, dtype_code, plain_function, ptr, sm_count
 
-EPI_BF16, EPI_F32, EPI_ACCUM, EPI_GATED, EPI_CLAMPED = 0, 1, 2, 3, 4
+EPI_BF16, EPI_F32, EPI_ACCUM, EPI_GATED, EPI_CLAMPED, EPI_RELU2 = 0, 1, 2, 3, 4, 5
 
 _weight_maps: dict = {}
 MAX_PARTS = 16      # K ranges whose sums the reader adds
@@ -103,7 +103,7 @@ def choose_parts(m: int, n: int, k: int) -> tuple:
 def gemm(x: torch.Tensor, weight: torch.Tensor, bias, epi: int, out: torch.Tensor,
          n: int, dual_offset: int = 0, splits: int | None = None, parts: int = 1,
          clamp: tuple = (0.0, 0.0, 0.0)) -> torch.Tensor:
-    """`out` is written (EPI_BF16, EPI_F32, EPI_GATED) or added to (EPI_ACCUM); `n` is the
+    """`out` is written (EPI_BF16, EPI_F32, EPI_GATED, EPI_RELU2) or added to (EPI_ACCUM); `n` is the
     number of output columns (rows of `weight`, or half of them for EPI_GATED). With
     `parts` > 1 (EPI_F32, `out` [parts, M, n]) K is cut into that many ranges whose sums are
     left apart in `out[i]`, with the bias in `out[0]`. `clamp`: EPI_CLAMPED's (limit, alpha,

@@ -91,6 +91,17 @@ def gated_up(x: torch.Tensor, w_gate_up: torch.Tensor, clamp: tuple | None = Non
     return gated_silu(both) if clamp is None else clamped_act(both, *clamp)
 
 
+def dense_up(x: torch.Tensor, w_up: torch.Tensor) -> torch.Tensor:
+    """`max(x Wup^T, 0)^2` of x's type: one kernel with the activation in its epilogue where the
+    tensor-core kernel takes the operands, else the product followed by the activation kernel."""
+    from . import relu_squared
+    if x.shape[0] <= TC_MAX_TOKENS and gemm_tc.takes(x, w_up):
+        out = torch.empty((x.shape[0], w_up.shape[0]), dtype=torch.bfloat16, device=x.device)
+        return gemm_tc.gemm(x, w_up, None, gemm_tc.EPI_RELU2, out, w_up.shape[0])
+    up = linear(x, w_up, out_dtype=x.dtype)
+    return relu_squared(up, out=up)
+
+
 def per_head(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     """A product a head: `out[:, h] = x[:, h] weight[h]^T` for x [T, heads, K], weight [heads,
     N, K] (contiguous) and out [T, heads, N], both views with any strides between tokens and

@@ -47,15 +47,17 @@ def router_logits(h: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 
 def route(logits: torch.Tensor, experts: int, top: int, identity: int = 0,
           softmax: bool = False, bias: torch.Tensor | None = None, groups: int = 1,
-          keep_groups: int = 1, renormalize: bool = False) -> Routing:
+          keep_groups: int = 1, renormalize: bool = False, group_top: int = 1,
+          scale: float = 1.0) -> Routing:
     """logits: fp32 [T, >= experts + identity]; the `top` largest scores among the first
     `experts + identity` columns a row. The score is the sigmoid of the logit, or with
     `softmax` the softmax over those columns; `bias` (fp32 [experts + identity]) is added for
     the choice only. A choice among the last `identity` columns is an identity expert: it gets
     no row in the grouped products, and `combine` adds the token's input times its weight.
     `groups` g (up to 64): the columns form g equal groups of neighbours, and only those of the
-    `keep_groups` groups with the largest best score can be chosen. `renormalize`: the weights
-    are the chosen scores divided by (their sum + 1e-20)."""
+    `keep_groups` groups with the largest best score (`group_top` 2: the largest sum of their two
+    best) can be chosen. `renormalize`: the weights are the chosen scores divided by (their sum +
+    1e-20). `scale` multiplies the weights."""
     require_cuda(logits, bias)
     outputs = experts + identity
     _check(logits.dtype == torch.float32 and logits.dim() == 2 and logits.stride(1) == 1
@@ -80,12 +82,12 @@ def route(logits: torch.Tensor, experts: int, top: int, identity: int = 0,
     if 0 < tokens <= ROUTE_IN_ONE_BLOCK:
         call("sakv_moe_route_plan", ptr(logits), logits.stride(0), outputs, top, ptr(r.chosen),
              ptr(r.weights), ptr(r.rank), tokens, experts, int(bool(softmax)), ptr(bias),
-             int(groups), int(keep_groups), int(bool(renormalize)),
+             int(groups), int(keep_groups), int(bool(renormalize)), int(group_top), float(scale),
              ptr(r.offsets), ptr(r.tile_expert), ptr(r.tile_row), ptr(r.n_tiles), r.max_tiles)
         return r
     call("sakv_moe_route", ptr(logits), logits.stride(0), outputs, top, ptr(r.chosen),
          ptr(r.weights), ptr(counts), ptr(r.rank), tokens, experts, int(bool(softmax)), ptr(bias),
-         int(groups), int(keep_groups), int(bool(renormalize)))
+         int(groups), int(keep_groups), int(bool(renormalize)), int(group_top), float(scale))
     call("sakv_moe_plan", ptr(counts), ptr(r.offsets), ptr(r.tile_expert), ptr(r.tile_row),
          ptr(r.n_tiles), experts, r.max_tiles)
     return r

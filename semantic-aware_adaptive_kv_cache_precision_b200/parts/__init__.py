@@ -21,10 +21,13 @@ from .selective_scan import SelectiveScanMixer
 from .output_norm import OutputNormBlock
 from .post_norm import PostNormBlock, PostNormUpdate
 from .dual_scan import DualScanMixer
+from .gated_delta import GatedDeltaMixer
+from .parallel_block import ParallelBlock
 
 __all__ = ["Part", "build_part", "register_part", "RMSNorm", "RotaryHalf", "RotaryInterleaved", "NoPosition",
            "GQAAttention", "GatedMLP", "DenseMLP", "PreNormBlock", "DeltaRuleMixer",
            "LogDistanceAttention", "StreamBlock", "StreamUpdate", "LayerNorm", "LatentAttention",
            "DifferentialAttention", "RoutedExperts", "SandwichBlock", "NormedUpdate",
            "WindowSinkAttention", "DecayAttention", "ParallelMixer", "SelectiveScanMixer",
-           "OutputNormBlock", "PostNormBlock", "PostNormUpdate", "DualScanMixer"]
+           "OutputNormBlock", "PostNormBlock", "PostNormUpdate", "DualScanMixer",
+           "GatedDeltaMixer", "ParallelBlock"]

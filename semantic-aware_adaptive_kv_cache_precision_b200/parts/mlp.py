@@ -58,13 +58,16 @@ class GatedMLP(Part):
 
 
 class DenseMLP(Part):
-    """Dense feed-forward without a gate, `down(act(up(h)))`, with the tanh form of GELU
-    (fp32 inside, one rounding at its store); tensors `up` and `down`."""
+    """Dense feed-forward without a gate, `down(act(up(h)))`, with the tanh form of GELU or the
+    square of relu (fp32 inside, one rounding at its store); tensors `up` and `down`."""
+
+    kernel_libraries = ("elementwise",)
 
     def __init__(self, spec, prefix, mode):
         super().__init__(spec, prefix, mode)
-        if spec.activation != "gelu_tanh":
-            raise ValueError(f"activation {spec.activation!r}: only 'gelu_tanh' is built")
+        if spec.activation not in ("gelu_tanh", "relu_squared"):
+            raise ValueError(f"activation {spec.activation!r}: 'gelu_tanh' and 'relu_squared' are "
+                             "built")
 
     def tensor_decls(self):
         s, p = self.spec, self.prefix
@@ -75,14 +78,20 @@ class DenseMLP(Part):
         self.w_up = arena.view(self.prefix + "up")
         self.w_down = arena.view(self.prefix + "down")
 
+    def _act(self, h):
+        if self.spec.activation == "relu_squared":
+            return ops.dense_up(h, self.w_up)
+        return ops.gelu_tanh(ops.linear(h, self.w_up, out_dtype=self.act_dtype))
+
     def produce(self, h, step):
         """The feed-forward's output, fp32 [T, hidden]."""
-        act = ops.gelu_tanh(ops.linear(h, self.w_up, out_dtype=self.act_dtype))
-        return ops.linear(act, self.w_down, out_dtype=torch.float32)
+        return ops.linear(self._act(h), self.w_down, out_dtype=torch.float32)
 
-    def forward(self, h, step, residual):
-        ops.linear(ops.gelu_tanh(ops.linear(h, self.w_up, out_dtype=self.act_dtype)),
-                   self.w_down, accumulate_into=residual)
+    can_defer = True
+
+    def forward(self, h, step, residual, defer=False):
+        out = ops.linear(self._act(h), self.w_down, accumulate_into=residual, may_defer=defer)
+        return out.delta if isinstance(out, ops.Deferred) else None
 
 
 register_part("gated_mlp", GatedMLP)

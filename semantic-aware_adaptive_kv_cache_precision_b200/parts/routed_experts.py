@@ -8,9 +8,9 @@
         (or the plain gated form: limit infinite, alpha 1, and 0 in the place of the 1)
     out = sum_chosen expert_e(s_e h)  +  sigmoid(h Wsg^T) * shared(h)
 
-The outputs may form groups of which only the best few are open to a token. The chosen scores
-are used as they are (or divided by their sum with `renormalize`) and
-multiply the expert's INPUT (`weight_input`) or its output. Everything stays on the device:
+The outputs may form groups of which only the best few (by their largest score, or the sum of
+their two largest) are open to a token. The chosen scores are used as they are (or divided by
+their sum with `renormalize`), times `scale`, and multiply the expert's INPUT (`weight_input`) or its output. Everything stays on the device:
 the router's product runs in fp32 on the step's tokens, a kernel chooses and counts, the
 tokens' rows are sorted by expert, and two grouped products (gate and up with the activation
 in the epilogue, then down) run over tiles of one expert's rows each (`csrc/moe.cu`). The
@@ -41,6 +41,8 @@ class RoutedExperts(Part):
                 or self.outputs // spec.groups * spec.keep_groups < spec.top:
             raise ValueError(f"{spec.groups} groups of which {spec.keep_groups} stay open do not "
                              f"fit {self.outputs} outputs and top {spec.top}")
+        if spec.group_top not in (1, 2):
+            raise ValueError(f"group_top {spec.group_top}: 1 and 2 are built")
         if spec.experts < 1 or spec.identity < 0 or spec.top > self.outputs \
                 or self.outputs > 1024 or spec.top > 32:
             raise ValueError("the router takes up to 1024 outputs (experts and identity "
@@ -100,7 +102,8 @@ class RoutedExperts(Part):
         s = self.spec
         logits = mixture.router_logits(h, self.w_route)
         routing = mixture.route(logits, s.experts, s.top, s.identity, s.score == "softmax",
-                                self.correction, s.groups, s.keep_groups, s.renormalize)
+                                self.correction, s.groups, s.keep_groups, s.renormalize,
+                                s.group_top, s.scale)
         # (a checkpoint stored in 32 bits keeps its matrices so: the experts then run in 32 bits)
         rows = mixture.gather_rows(h if h.dtype == self.w_gate.dtype else h.to(self.w_gate.dtype),
                                    routing, s.weight_input)

@@ -7,6 +7,7 @@ logit a head in the softmax's denominator (`WindowSinkAttentionSpec`):
     q <- q * temperature(position), where there is one
     the first `rotary_dim` numbers of every head of q and k turned by the position
     s_ij = q_i . k_j * scale  for  j <= i  and  (i - j < window  or  j < keep_first)
+    s_ij <- softcap * tanh(s_ij / softcap),  s_ij <- s_ij - slope[h] * (i - j)    (where given)
     a_i = sum_j exp(s_ij) v_j / (sum_j exp(s_ij) + exp(sink[h]))
     out = Wo [out_scale * a * sigmoid(h Wg^T)]         (the gate, element by element, if there is one)
 
@@ -14,6 +15,10 @@ The fused projection leaves fp32 (its accumulator, unrounded); the two norms, th
 the cache write are one kernel (`csrc/qk_prepare.cu`); scores, softmax weights, the sink and the
 weighted sums are fp32 in both modes (`csrc/attention_distance.cu`). The cache keeps the blocks
 of the first `keep_first` positions for as long as the sequence lives (`KVNeed.keep_first`).
+
+A layer without projections of its own for keys and values (`own_kv` False) makes queries only and
+reads the cache entry of the layer whose keys and values it uses (its layer call names that
+entry; the layer that owns it ran earlier in the same step).
 
 The part is a mixer of its own (`produce`) and a branch of a `ParallelMixer` (`input_rows`,
 `input_decls`, `input_bias`, `mix`, `w_o`).
@@ -44,8 +49,13 @@ class WindowSinkAttention(Part):
         if s.keep_first and not s.window:
             raise ValueError("keep_first goes with a window")
         self.q_cols = s.heads * s.head_dim
-        self.k_cols = s.kv_heads * s.head_dim
-        self.v_cols = s.kv_heads * s.value_dim
+        if s.qk_norm == "whole" and not s.own_kv:
+            raise ValueError("qk_norm 'whole' is not built for a layer without keys of its own")
+        if s.slopes is not None and len(s.slopes) != s.heads:
+            raise ValueError("slopes: one number a head")
+        self.k_cols = s.kv_heads * s.head_dim if s.own_kv else 0
+        self.v_cols = s.kv_heads * s.value_dim if s.own_kv else 0
+        self.slopes = None
         self.position = None if s.position is None else build_part(s.position, prefix, mode)
         self.sink = self.temperature = None
         self.g_cols = s.heads * s.value_dim if s.gate else 0
@@ -57,7 +67,9 @@ class WindowSinkAttention(Part):
         return self.q_cols + self.k_cols + self.v_cols + self.g_cols
 
     def _inputs(self):
-        rows = (("q", self.q_cols), ("k", self.k_cols), ("v", self.v_cols))
+        rows = (("q", self.q_cols),)
+        if self.spec.own_kv:
+            rows += (("k", self.k_cols), ("v", self.v_cols))
         return rows + (("g", self.g_cols),) if self.g_cols else rows
 
     def input_decls(self, group):
@@ -104,6 +116,7 @@ class WindowSinkAttention(Part):
         `offset` on) to the input of `w_o`: [T, heads * value_dim] of the activations' type,
         `out_scale` included."""
         s = self.spec
+        write_cache = write_cache and s.own_kv
         cos = sin = None
         if self.position is not None:
             if step.max_position >= self.position.cos.shape[0]:
@@ -121,7 +134,8 @@ class WindowSinkAttention(Part):
             q.view(q.shape[0], s.heads, s.head_dim), view.keys, view.values, step.positions,
             step.token_seq, view.block_table, s.heads, s.head_dim, s.value_dim, s.scale,
             window=s.window, keep_first=s.keep_first if s.window else 0, sink=self.sink,
-            out_scale=s.out_scale, elem_gate=gate, **self._decode_form(step)).view(q.shape[0], -1)
+            out_scale=s.out_scale, elem_gate=gate, softcap=s.softcap, linear_slopes=self.slopes,
+            **self._decode_form(step)).view(q.shape[0], -1)
 
     def _temperature(self, step):
         if self.temperature is not None and step.max_position >= self.temperature.numel():
@@ -159,6 +173,8 @@ class WindowSinkAttention(Part):
     def prepare(self, device, max_positions):
         if self.position is not None:
             self.position.prepare(device, max_positions)
+        if self.spec.slopes is not None:
+            self.slopes = torch.tensor(self.spec.slopes, dtype=torch.float32, device=device)
         t = self.spec.q_temp
         if t is not None:       # worked out in float64, kept in fp32
             p = torch.arange(max_positions, dtype=torch.float64)
