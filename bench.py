@@ -395,6 +395,23 @@ def kernel_case(name: str) -> int:
         step = SimpleNamespace(cu_seqlens=i32([0, n]), slots=i32([0]), sequences=1, max_new=n)
         run = lambda i: ops.dual_scan(xbc, 0, heads * vdim, heads * vdim + ns, dt, bias, a, skip,
                                       heads, 1, ns, vdim, state, step, run=64)
+    elif name == "gated_delta_4096":
+        # the gated delta rule over one prompt of 4,096 tokens at the `2k` size of `--design gozolix`
+        # (16 heads of 128 x 128, q and k of 8), four tokens at a time: about 250 MB
+        from types import SimpleNamespace
+        n, heads, kv_heads, dim, vdim = 4096, 16, 8, 128, 128
+        channels = 2 * kv_heads * dim + heads * vdim
+        proj = torch.randn(n, channels + heads * vdim + 2 * heads, device=dev)
+        conv = torch.randn(channels, 4, device=dev).to(torch.bfloat16)
+        a, bias = -torch.rand(heads, device=dev) - 0.1, torch.full((heads,), -3.0, device=dev)
+        conv_state = torch.zeros(1, 3, channels, device=dev)
+        state = torch.zeros(1, heads, vdim, dim, device=dev)
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        step = SimpleNamespace(cu_seqlens=i32([0, n]), slots=i32([0]), sequences=1, max_new=n)
+        run = lambda i: ops.gated_delta(proj, channels + heads * vdim,
+                                        channels + heads * vdim + heads, conv, a, bias, conv_state,
+                                        state, step, heads, kv_heads, dim, vdim, dim ** -0.5, 1e-6,
+                                        by_groups=True)
     else:
         raise SystemExit(f"unknown kernel case {name}")
     for i in range(4):
@@ -826,6 +843,127 @@ def felovik_rates(size, kernels, gsize, batch, context, tokens, hbm) -> dict:
     return out
 
 
+#: layer sizes for `--design gozolix`: (width; the recurrence's heads, q/k heads, dim, vdim and taps;
+#: attention heads / kv heads x (dim, vdim); dense feed-forward; experts, chosen, their width, groups
+#: of experts, how many stay open, the shared expert's width)
+GOZOLIX_SIZES = {
+    "1k": dict(width=1024, delta=(16, 8, 64, 64, 4), attention=(8, 2, 128, 128), ff=4096,
+               experts=(16, 2, 1024, 4, 2, 1024), vocab=32768, layers=6),
+    "2k": dict(width=2048, delta=(16, 8, 128, 128, 4), attention=(16, 4, 128, 128), ff=8192,
+               experts=(32, 4, 1024, 8, 4, 2048), vocab=32768, layers=6),
+}
+
+
+def gozolix_configs(size: dict) -> dict:
+    """Configs by label: Gozolix (two delta layers, then one of attention, twice; the second
+    attention layer reads the first one's keys and values) with dense feed-forwards only and with
+    experts in two layers of three; the Tebonex config with the same order of layers, heads of equal
+    number and sizes in both mixers, attention over every earlier key and a dense feed-forward of
+    equal size: the library's other design with a delta rule and a distance penalty; and the
+    Felovik config with equal experts."""
+    heads, kv_heads, dim, vdim = size["attention"]
+    dheads, dkv, ddim, dvdim, taps = size["delta"]
+    experts, top, eff, count, keep, shared = size["experts"]
+    delta = {"heads": dheads, "kv_heads": dkv, "dim": ddim, "vdim": dvdim, "conv": taps}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim,
+                 "scale": dim ** -0.5}
+    own = dict(attention, softcap=50.0, q_temp={"coef": 0.1, "every": 1024})
+    dense = {"kind": "dense", "ff": size["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": eff}, "shared": {"ff": shared},
+           "router": {"experts": experts, "top": top, "scale": 2.5,
+                      "groups": {"count": count, "keep": keep}}}
+    common = {"vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-6},
+              "initializer_range": 0.02}
+
+    def gozolix(mlps):
+        layers = []
+        for i, m in enumerate(mlps):
+            if i % 3 < 2:
+                layers.append({"type": "delta", "mixer": delta, "mlp": m})
+            else:
+                layers.append({"type": "attention", "mlp": m,
+                               "mixer": own if i < 3 else dict(own, kv_from=2)})
+        return {"architecture": "Gozolix", **common, "layers": layers,
+                "embedding": {"scale": 1.0, "bigram": {"buckets": 32749, "mul_prev": 31,
+                                                       "mul_cur": 7}}}
+
+    other, _ = design_configs(dict(size, delta=(dheads, ddim), streams=None, window=None,
+                                   attention=(heads, kv_heads, dim)))
+    del other["streams"]
+    fsize = FELOVIK_SIZES["1k"]
+    felovik = felovik_configs(dict(fsize, width=size["width"], ff=size["ff"],
+                                   experts=size["experts"][:5], vocab=size["vocab"],
+                                   attention=size["attention"]))["felovik_experts"]
+    n = size["layers"]
+    return {"tebonex": other, "gozolix_dense": gozolix([dense] * n),
+            "gozolix_experts": gozolix([dense if i % 3 == 0 else moe for i in range(n)]),
+            "felovik": felovik}
+
+
+def gozolix_rates(size, kernels, batch, context, tokens, hbm) -> dict:
+    """What the designs' own kernels must move or compute in the timed steps, against the
+    measured peaks. `kernels`: kernel times by label (`gozolix_configs`)."""
+    heads, kv_heads, dim, vdim = size["attention"]
+    dheads, dkv, ddim, dvdim, taps = size["delta"]
+    experts, top, eff, _, _, shared = size["experts"]
+    n, width = size["layers"], size["width"]
+    n_delta = sum(1 for i in range(n) if i % 3 < 2)
+    n_moe = sum(1 for i in range(n) if i % 3)
+    channels, inner = 2 * dkv * ddim + dheads * dvdim, dheads * dvdim
+    g, e, t, f = (kernels[k] for k in ("gozolix_dense", "gozolix_experts", "tebonex", "felovik"))
+
+    def of_hbm(nbytes, us):
+        return round(nbytes / (us * 1e-6) / 1e9 / hbm, 3) if us else None
+
+    def tflops(flops, us):
+        return round(flops / (us * 1e-6) / 1e12, 2) if us else None
+
+    def total(times, *names):
+        return sum(times.get(k, 0.0) for k in names)
+
+    out = {}
+    # the recurrence over a prompt: a state element's decay, the sum along the key, the update and
+    # the sum along the query, 7 operations a token
+    ops_ = 7.0 * tokens * dheads * ddim * dvdim * n_delta
+    out["delta_scan_prefill_tflops_fp32"] = tflops(ops_, g["prefill"].get("delta_scan"))
+    out["delta_all_prefill_tflops_fp32"] = tflops(
+        ops_, total(g["prefill"], "delta_inputs", "delta_scan", "conv_state", "norm_gate"))
+    out["tebonex_delta_rule_prefill_tflops_fp32"] = tflops(ops_, t["prefill"].get("delta_rule"))
+    out["delta_inputs_prefill_of_measured_hbm"] = of_hbm(
+        tokens * channels * 8 * n_delta, g["prefill"].get("delta_inputs"))
+    out["norm_gate_prefill_of_measured_hbm"] = of_hbm(
+        tokens * inner * 10 * n_delta, g["prefill"].get("norm_gate"))
+    moved = batch * dheads * ddim * dvdim * 4 * 2 * n_delta            # the state, in and out
+    out["delta_scan_decode_of_measured_hbm"] = of_hbm(moved, g["decode"].get("delta_scan"))
+    out["delta_all_decode_of_measured_hbm"] = of_hbm(
+        moved, total(g["decode"], "delta_inputs", "delta_scan", "norm_gate"))
+    out["tebonex_delta_rule_decode_of_measured_hbm"] = of_hbm(moved, t["decode"].get("delta_rule"))
+    flops = 2.0 * heads * (dim + vdim) * tokens * (tokens + 1) / 2 * (n - n_delta)
+    read = batch * context * kv_heads * (dim + vdim) * 2 * (n - n_delta)
+    for label, times, name in (("", g, "cached_attention"), ("tebonex_", t, "distance_attention")):
+        out[label + "attention_prefill_tflops_fp32"] = tflops(flops, times["prefill"].get(name))
+        out[label + "attention_decode_of_measured_hbm"] = of_hbm(read, times["decode"].get(name))
+    out["relu_squared_prefill_of_measured_hbm"] = of_hbm(
+        tokens * size["ff"] * 4 * n, g["prefill"].get("relu_squared"))
+    out["tebonex_gelu_prefill_of_measured_hbm"] = of_hbm(
+        tokens * size["ff"] * 4 * n, t["prefill"].get("gelu_tanh"))
+    # the embedding: two bf16 rows in, one fp32 row out (Tebonex: one row in)
+    out["embed_pairs_prefill_of_measured_hbm"] = of_hbm(tokens * width * 8,
+                                                        g["prefill"].get("embed_pairs"))
+    out["tebonex_embed_prefill_of_measured_hbm"] = of_hbm(tokens * width * 6,
+                                                          t["prefill"].get("embed"))
+    for label, times, layers in (("", e, n_moe), ("felovik_", f, n_moe)):
+        out[label + "experts_prefill_tflops_bf16"] = tflops(
+            6.0 * tokens * top * eff * width * layers, times["prefill"].get("moe_product"))
+        out[label + "experts_decode_of_measured_hbm"] = of_hbm(
+            min(batch * top, experts) * 3 * eff * width * 2 * layers,
+            times["decode"].get("moe_product"))
+        out[label + "route_us"] = {w: round(total(times[w], "moe_logits", "moe_route", "moe_plan",
+                                                  "moe_route_plan"), 1)
+                                   for w in ("prefill", "decode")}
+    return out
+
+
 def design_configs(size: dict) -> tuple:
     """(Tebonex config, the Qwen2 config of equal width, depth, heads and feed-forward)."""
     heads, kv_heads, dim = size["attention"]
@@ -833,7 +971,9 @@ def design_configs(size: dict) -> tuple:
     for i in range(size["layers"]):
         if i % 3 == 2:
             mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim,
-                     "scale": dim ** -0.5, "mask": {"size": size["window"]}}
+                     "scale": dim ** -0.5}
+            if size["window"] is not None:
+                mixer["mask"] = {"size": size["window"]}
             kind = "attention"
         else:
             mixer = {"heads": size["delta"][0], "dim": size["delta"][1], "decay_rank": 64}
@@ -1006,6 +1146,34 @@ def design_arm(args) -> int:
                           "batch": batch, "context": context, "prefill_tokens": tokens, "steps": K,
                           "warmup": W, "peaks": pk, "sizes": rows}))
         return 0
+    if args.design == "gozolix":
+        for name in sizes:
+            size = GOZOLIX_SIZES[name]
+            row = {"size": name, **{k: size[k] for k in ("width", "layers", "ff", "attention",
+                                                         "delta", "experts")}}
+            kernels = {}
+            for label, config in gozolix_configs(size).items():
+                engine, slots, prompt, out = measure(config)
+                row[label] = out
+                engine.close(slots)
+                engine.release()
+                del engine
+                torch.cuda.empty_cache()
+                engine, slots, prompt, _ = measure(config, graphs=False)
+                row[label + "_kernels_us"] = kernels[label] = kernel_times(engine, slots, prompt)
+                engine.close(slots)
+                engine.release()
+                del engine
+                torch.cuda.empty_cache()
+            row["kernel_rates"] = gozolix_rates(size, kernels, batch, context, tokens, hbm)
+            rows.append(row)
+        print(json.dumps({"design": "gozolix", "beside": "tebonex of equal width, depth, order of "
+                          "layers, heads of both mixers and feed-forward size, attention without "
+                          "a window; felovik for the experts", "dtype": "bf16",
+                          "data": "synthetic (random weights and tokens; weights larger than L2)",
+                          "batch": batch, "context": context, "prefill_tokens": tokens, "steps": K,
+                          "warmup": W, "peaks": pk, "sizes": rows}))
+        return 0
     if args.design == "felovik":
         for name in sizes:
             size, gsize = FELOVIK_SIZES[name], GESUVIK_SIZES[name]
@@ -1120,7 +1288,8 @@ def design_arm(args) -> int:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=["tebonex", "venanex", "zodirax", "gesuvik", "felovik"],
+    ap.add_argument("--design", default=None, choices=["tebonex", "venanex", "zodirax", "gesuvik", "felovik",
+                                                    "gozolix"],
                     help="instead of the default workload: the named design at layer sizes "
                          "that resemble real models, beside the Qwen2 decoder of equal size")
     ap.add_argument("--design-sizes", default="1k,2k", help="which of: " + ", ".join(DESIGN_SIZES))

@@ -69,29 +69,37 @@ struct DeltaInputs {
 };
 
 // silu of the convolution of one channel for the group's `m` tokens; token tt is number i0 + tt of
-// its sequence's part in this step. `move`: the part is this one token, and the channel's running
-// inputs go up by one place.
-template <typename W>
-__device__ __forceinline__ void conv_channel(const DeltaInputs<W>& p, const float* part, float* old,
-                                             int c, int i0, int m, float (&y)[kGroup]) {
-  const int keep = p.taps - 1;
+// its sequence's part in this step. Inputs before the part come from the sequence's running ones.
+// TAPS: the taps as a compile-time number, so that the window of inputs is read once for all four
+// tokens (0: any number). The products are added oldest first either way.
+template <int TAPS, typename W>
+__device__ __forceinline__ void conv_channel(const DeltaInputs<W>& p, const float* __restrict__ part,
+                                             const float* __restrict__ old, int c, int i0, int m,
+                                             float (&y)[kGroup]) {
+  const int taps = TAPS > 0 ? TAPS : p.taps, keep = taps - 1;
+  auto input = [&](int at) {                           // input number `at` of this step's part
+    return at >= 0 ? __ldg(part + (long long)at * p.stride + c)
+                   : __ldg(old + (long long)(keep + at) * p.channels + c);
+  };
 #pragma unroll
   for (int tt = 0; tt < kGroup; ++tt) y[tt] = 0.f;
-  for (int j = 0; j < p.taps; ++j) {
-    const float w = widen(p.conv[(long long)c * p.taps + j]);
+  if constexpr (TAPS > 0) {
+    float x[TAPS - 1 + kGroup], w[TAPS];
 #pragma unroll
-    for (int tt = 0; tt < kGroup; ++tt) {
-      if (tt >= m) continue;
-      const int at = i0 + tt - (keep - j);             // the input's number in this step's part
-      const float x = at >= 0 ? part[(long long)at * p.stride + c]
-                              : old[(long long)(keep + at) * p.channels + c];
-      y[tt] = fmaf(x, w, y[tt]);
+    for (int i = 0; i < TAPS - 1 + kGroup; ++i) x[i] = i < keep + m ? input(i0 - keep + i) : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = widen(p.conv[(long long)c * TAPS + j]);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int tt = 0; tt < kGroup; ++tt) y[tt] = fmaf(x[tt + j], w[j], y[tt]);
+  } else {
+    for (int j = 0; j < taps; ++j) {
+      const float w = widen(p.conv[(long long)c * taps + j]);
+#pragma unroll
+      for (int tt = 0; tt < kGroup; ++tt)
+        if (tt < m) y[tt] = fmaf(input(i0 + tt - (keep - j)), w, y[tt]);
     }
-  }
-  if (p.move_state && keep > 0) {
-    for (int j = 0; j + 1 < keep; ++j)
-      old[(long long)j * p.channels + c] = old[(long long)(j + 1) * p.channels + c];
-    old[(long long)(keep - 1) * p.channels + c] = part[c];
   }
 #pragma unroll
   for (int tt = 0; tt < kGroup; ++tt) y[tt] = silu(y[tt]);
@@ -100,7 +108,7 @@ __device__ __forceinline__ void conv_channel(const DeltaInputs<W>& p, const floa
 // Grid: (units of warps, sequences). A group's units are its kv_heads (q and k of one head, with
 // the decays, betas and group numbers of the heads that read it), then runs of 32 * PER channels
 // of v. PER * 32 >= dim.
-template <int PER, typename W>
+template <int PER, int TAPS, typename W>
 __global__ void __launch_bounds__(128) delta_inputs_kernel(const DeltaInputs<W> p) {
   let_next_kernel_start();
   wait_for_previous_kernel();
@@ -114,59 +122,66 @@ __global__ void __launch_bounds__(128) delta_inputs_kernel(const DeltaInputs<W> 
   if (i0 >= n) return;
   const int m = n - i0 < kGroup ? n - i0 : kGroup;
   const float* part = p.proj + (long long)first * p.stride;
-  float* old = p.conv_state + (long long)p.slots[b] * (p.taps - 1) * p.channels;
-  float* out = p.prepared + (long long)(first + i0) * p.channels;
+  const float* old = p.conv_state + (long long)p.slots[b] * (p.taps - 1) * p.channels;
+  float* __restrict__ out = p.prepared + (long long)(first + i0) * p.channels;
   const int qk = p.kv_heads * p.dim;
-  float y[kGroup];
 
   if (unit >= p.kv_heads) {                            // values: the convolution is all
     const int c0 = (unit - p.kv_heads) * 32 * PER;
+    float y[PER][kGroup];
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
       const int c = c0 + lane + 32 * i;
-      if (c >= v_width) continue;
-      conv_channel(p, part, old, 2 * qk + c, i0, m, y);
+      if (c < v_width) conv_channel<TAPS>(p, part, old, 2 * qk + c, i0, m, y[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int c = c0 + lane + 32 * i;
 #pragma unroll
       for (int tt = 0; tt < kGroup; ++tt)
-        if (tt < m) out[(long long)tt * p.channels + 2 * qk + c] = y[tt];
+        if (tt < m && c < v_width) out[(long long)tt * p.channels + 2 * qk + c] = y[i][tt];
     }
     return;
   }
 
-  float q[kGroup][PER], k[kGroup][PER];
-  float qq[kGroup] = {}, kk[kGroup] = {};
+  float q[PER][kGroup], k[PER][kGroup];
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i, c = unit * p.dim + e;
 #pragma unroll
-    for (int tt = 0; tt < kGroup; ++tt) q[tt][i] = k[tt][i] = 0.f;
-    if (e >= p.dim) continue;
-    conv_channel(p, part, old, c, i0, m, y);
-#pragma unroll
-    for (int tt = 0; tt < kGroup; ++tt)
-      if (tt < m) { q[tt][i] = y[tt]; qq[tt] = fmaf(y[tt], y[tt], qq[tt]); }
-    conv_channel(p, part, old, qk + c, i0, m, y);
-#pragma unroll
-    for (int tt = 0; tt < kGroup; ++tt)
-      if (tt < m) { k[tt][i] = y[tt]; kk[tt] = fmaf(y[tt], y[tt], kk[tt]); }
+    for (int tt = 0; tt < kGroup; ++tt) q[i][tt] = k[i][tt] = 0.f;
+    if (e < p.dim) {
+      conv_channel<TAPS>(p, part, old, c, i0, m, q[i]);
+      conv_channel<TAPS>(p, part, old, qk + c, i0, m, k[i]);
+    }
   }
 #pragma unroll
   for (int tt = 0; tt < kGroup; ++tt) {
-    const float rq = p.q_scale / sqrtf(warp_sum(qq[tt]) + p.unit_eps);
-    const float rk = 1.f / sqrtf(warp_sum(kk[tt]) + p.unit_eps);
+    if (tt >= m) {                                     // (a token that is missing: zeros)
+#pragma unroll
+      for (int i = 0; i < PER; ++i) q[i][tt] = k[i][tt] = 0.f;
+    }
+    float qq = 0.f, kk = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      qq = fmaf(q[i][tt], q[i][tt], qq);
+      kk = fmaf(k[i][tt], k[i][tt], kk);
+    }
+    const float rq = p.q_scale / sqrtf(warp_sum(qq) + p.unit_eps);
+    const float rk = 1.f / sqrtf(warp_sum(kk) + p.unit_eps);
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
       const int e = lane + 32 * i;
-      q[tt][i] *= rq;
-      k[tt][i] *= rk;
+      q[i][tt] *= rq;
+      k[i][tt] *= rk;
       if (tt < m && e < p.dim) {
         float* row = out + (long long)tt * p.channels + unit * p.dim + e;
-        row[0] = q[tt][i];
-        row[qk] = k[tt][i];
+        row[0] = q[i][tt];
+        row[qk] = k[i][tt];
       }
     }
   }
-  // k_j . q_i and k_j . k_i of the group (zeros for the tokens it lacks)
+  // k_j . q_i and k_j . k_i of the group
   float kq[kGroup][kGroup] = {}, kkg[kGroup][kGroup] = {};
   if (p.coef != nullptr) {
 #pragma unroll
@@ -176,60 +191,138 @@ __global__ void __launch_bounds__(128) delta_inputs_kernel(const DeltaInputs<W> 
         float s = 0.f, r = 0.f;
 #pragma unroll
         for (int e = 0; e < PER; ++e) {
-          s = fmaf(k[j][e], q[i][e], s);
-          if (j < i) r = fmaf(k[j][e], k[i][e], r);
+          s = fmaf(k[e][j], q[e][i], s);
+          if (j < i) r = fmaf(k[e][j], k[e][i], r);
         }
         kq[i][j] = warp_sum(s);
         if (j < i) kkg[i][j] = warp_sum(r);
       }
   }
-  const int per = p.heads / p.kv_heads;
-  for (int x = lane; x < per; x += 32) {
-    const int h = unit * per + x;
-    float log_g[kGroup], beta[kGroup];
-#pragma unroll
-    for (int tt = 0; tt < kGroup; ++tt) {
-      log_g[tt] = beta[tt] = 0.f;
-      if (tt >= m) continue;
-      const float* row = part + (long long)(i0 + tt) * p.stride;
-      log_g[tt] = softplus(row[p.a_off + h] + p.dt_bias[h]) * p.a[h];
-      beta[tt] = 1.f / (1.f + expf(-row[p.b_off + h]));
-      float* to = p.gates + ((long long)(first + i0 + tt) * p.heads + h) * 2;
-      to[0] = expm1f(log_g[tt]);
-      to[1] = beta[tt];
-    }
-    if (p.coef == nullptr) continue;
-    float* to = p.coef + ((first_group(p.cu_seqlens, b) + group) * p.heads + h) * kCoef;
-    float since = 0.f;                                  // the logarithm of c_i
-#pragma unroll
-    for (int i = 0; i < kGroup; ++i) {
-      since += log_g[i];
-      const float c = expf(since);
-      to[kBeta + i] = beta[i];
-      to[kBetaC + i] = beta[i] * c;
-      to[kC + i] = c;
-      float between = 0.f;                              // the logarithm of c_i / c_j
-#pragma unroll
-      for (int j = kGroup - 1; j >= 0; --j) {
-        if (j > i) {
-          to[kOut + 4 * i + j] = 0.f;
-          continue;
-        }
-        if (j < i) between += log_g[j + 1];
-        const float d = expf(between);
-        to[kOut + 4 * i + j] = d * kq[i][j];
-        if (j < i) to[kSolve + i * (i - 1) / 2 + j] = beta[i] * d * kkg[i][j];
+  // a lane a (head, token of the group)
+  const int per = p.heads / p.kv_heads, i = lane & 3;
+  for (int x0 = 0; x0 < per; x0 += 8) {
+    const int x = x0 + (lane >> 2);
+    const bool live = x < per;
+    const int h = unit * per + (live ? x : 0);
+    float log_g = 0.f, beta = 0.f;
+    if (i < m) {
+      const float* row = part + (long long)(i0 + i) * p.stride;
+      log_g = softplus(row[p.a_off + h] + p.dt_bias[h]) * p.a[h];
+      beta = 1.f / (1.f + expf(-row[p.b_off + h]));
+      if (live) {
+        float* to = p.gates + ((long long)(first + i0 + i) * p.heads + h) * 2;
+        to[0] = expm1f(log_g);
+        to[1] = beta;
       }
     }
-    to[kFade] = expm1f(since);
-    to[kFade + 1] = 0.f;
-    float rest = 0.f;                                   // (a token that is missing fades nothing)
+    if (p.coef == nullptr) continue;
+    float g[kGroup], since = 0.f, rest = 0.f, between = 0.f;
+#pragma unroll
+    for (int j = 0; j < kGroup; ++j) {
+      g[j] = __shfl_sync(0xffffffffu, log_g, (lane & ~3) + j);
+      if (j <= i) since += g[j];                        // the logarithm of c_i
+      else rest += g[j];                                // from token i to the group's end
+    }
+    if (!live) continue;
+    float* to = p.coef + ((first_group(p.cu_seqlens, b) + group) * p.heads + h) * kCoef;
+    const float c = expf(since);
+    to[kBeta + i] = beta;
+    to[kBetaC + i] = beta * c;
+    to[kC + i] = c;
+    to[kEnd + i] = expf(rest);
 #pragma unroll
     for (int j = kGroup - 1; j >= 0; --j) {
-      to[kEnd + j] = expf(rest);
-      rest += log_g[j];
+      if (j + 1 < kGroup && j < i) between += g[j + 1];  // the logarithm of c_i / c_j
+      float along_q = kq[0][j], along_k = 0.f;
+#pragma unroll
+      for (int r = 1; r < kGroup; ++r)
+        if (r == i) {
+          along_q = kq[r][j];
+          along_k = kkg[r][j];
+        }
+      const float d = expf(between);
+      to[kOut + 4 * i + j] = j <= i ? d * along_q : 0.f;
+      if (j < i) to[kSolve + i * (i - 1) / 2 + j] = beta * d * along_k;
+    }
+    if (i == kGroup - 1) {
+      to[kFade] = expm1f(since);
+      to[kFade + 1] = 0.f;
     }
   }
+}
+
+// The same for a step in which every sequence brings one token: a thread a channel, a block q and k
+// of one head (with its heads' decays and betas) or blockDim channels of v. Every sum has its terms
+// in the order of the kernel above. The running inputs go up by one place.
+template <typename W>
+__global__ void delta_inputs_step_kernel(const DeltaInputs<W> p) {
+  extern __shared__ float ys[];                        // [2 dim]
+  __shared__ float inv[2];
+  let_next_kernel_start();
+  wait_for_previous_kernel();
+  const int b = blockIdx.y, unit = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const long long t = p.cu_seqlens[b];
+  const int qk = p.kv_heads * p.dim, keep = p.taps - 1;
+  const float* row = p.proj + t * p.stride;
+  float* old = p.conv_state + (long long)p.slots[b] * keep * p.channels;
+  float* out = p.prepared + t * p.channels;
+  auto conv = [&](int c) {
+    constexpr int kMost = 7;                           // running inputs held in registers
+    const float now = row[c];
+    float y = 0.f;
+    if (keep <= kMost) {
+      float x[kMost + 1];
+#pragma unroll
+      for (int j = 0; j < kMost; ++j) x[j] = j < keep ? old[(long long)j * p.channels + c] : now;
+      x[kMost] = now;
+#pragma unroll
+      for (int j = 0; j < kMost + 1; ++j)
+        if (j <= keep) y = fmaf(x[j], widen(p.conv[(long long)c * p.taps + j]), y);
+      if (p.move_state) {
+#pragma unroll
+        for (int j = 0; j < kMost; ++j)
+          if (j < keep) old[(long long)j * p.channels + c] = x[j + 1];
+      }
+    } else {
+      for (int j = 0; j < keep; ++j)
+        y = fmaf(old[(long long)j * p.channels + c], widen(p.conv[(long long)c * p.taps + j]), y);
+      y = fmaf(now, widen(p.conv[(long long)c * p.taps + keep]), y);
+      if (p.move_state) {
+        for (int j = 0; j + 1 < keep; ++j)
+          old[(long long)j * p.channels + c] = old[(long long)(j + 1) * p.channels + c];
+        old[(long long)(keep - 1) * p.channels + c] = now;
+      }
+    }
+    return silu(y);
+  };
+  if (unit >= p.kv_heads) {
+    const int c = (unit - p.kv_heads) * blockDim.x + threadIdx.x;
+    if (c < p.heads * p.vdim) out[2 * qk + c] = conv(2 * qk + c);
+    return;
+  }
+  const int e = threadIdx.x;
+  const bool mine = e < 2 * p.dim, is_k = e >= p.dim;
+  const int c = (is_k ? qk - p.dim : 0) + unit * p.dim + e;
+  float y = 0.f;
+  if (mine) ys[e] = y = conv(c);
+  if (warp == 3) {                                     // (a block has four warps at least)
+    const int per = p.heads / p.kv_heads;
+    for (int x = lane; x < per; x += 32) {
+      const int h = unit * per + x;
+      float* to = p.gates + (t * p.heads + h) * 2;
+      to[0] = expm1f(softplus(row[p.a_off + h] + p.dt_bias[h]) * p.a[h]);
+      to[1] = 1.f / (1.f + expf(-row[p.b_off + h]));
+    }
+  }
+  __syncthreads();
+  if (warp < 2) {
+    float s = 0.f;
+    for (int i = lane; i < p.dim; i += 32) s = fmaf(ys[warp * p.dim + i], ys[warp * p.dim + i], s);
+    s = warp_sum(s);
+    if (lane == 0) inv[warp] = (warp == 0 ? p.q_scale : 1.f) / sqrtf(s + p.unit_eps);
+  }
+  __syncthreads();
+  if (mine) out[c] = y * inv[is_k];
 }
 
 __device__ __forceinline__ void copy16_async(float* dst, const float* src) {
@@ -562,20 +655,35 @@ int launch_scan(DeltaScan p, int sequences, int max_new, bool groups, cudaStream
 
 template <typename W>
 int launch_inputs(const DeltaInputs<W>& p, int sequences, int max_new, cudaStream_t stream) {
-#define SAKV_INPUTS(PER)                                                                         \
+  const long long v_width = (long long)p.heads * p.vdim;
+  if (max_new == 1 && p.coef == nullptr) {
+    const int threads = p.dim <= 64 ? 128 : (2 * p.dim + 31) / 32 * 32;
+    const long long units = p.kv_heads + (v_width + threads - 1) / threads;
+    if (units > 0x7fffffffLL) return cudaErrorInvalidValue;
+    return launch_overlapped(delta_inputs_step_kernel<W>, dim3((unsigned)units, (unsigned)sequences),
+                             dim3(threads), (size_t)2 * p.dim * sizeof(float), stream, 1, p);
+  }
+#define SAKV_INPUTS(PER, TAPS)                                                                   \
   do {                                                                                           \
-    const long long units = p.kv_heads + ((long long)p.heads * p.vdim + 32 * PER - 1) / (32 * PER); \
+    const long long units = p.kv_heads + (v_width + 32 * PER - 1) / (32 * PER);                  \
     const long long warps = units * ((max_new + kGroup - 1) / kGroup);                           \
     const long long blocks = (warps + 3) / 4;                                                    \
     if (blocks > 0x7fffffffLL) return cudaErrorInvalidValue;                                     \
-    return launch_overlapped(delta_inputs_kernel<PER, W>, dim3((unsigned)blocks, (unsigned)sequences), \
-                             dim3(128), 0, stream, 1, p);                                        \
+    return launch_overlapped(delta_inputs_kernel<PER, TAPS, W>,                                  \
+                             dim3((unsigned)blocks, (unsigned)sequences), dim3(128), 0, stream,  \
+                             1, p);                                                              \
   } while (0)
-  if (p.dim <= 32) SAKV_INPUTS(1);
-  if (p.dim <= 64) SAKV_INPUTS(2);
-  if (p.dim <= 128) SAKV_INPUTS(4);
-  if (p.dim <= 256) SAKV_INPUTS(8);
-  SAKV_INPUTS(16);
+  if (p.taps == 4) {                                   // (the usual width of these convolutions)
+    if (p.dim <= 32) SAKV_INPUTS(1, 4);
+    if (p.dim <= 64) SAKV_INPUTS(2, 4);
+    if (p.dim <= 128) SAKV_INPUTS(4, 4);
+    if (p.dim <= 256) SAKV_INPUTS(8, 4);
+  }
+  if (p.dim <= 32) SAKV_INPUTS(1, 0);
+  if (p.dim <= 64) SAKV_INPUTS(2, 0);
+  if (p.dim <= 128) SAKV_INPUTS(4, 0);
+  if (p.dim <= 256) SAKV_INPUTS(8, 0);
+  SAKV_INPUTS(16, 0);
 #undef SAKV_INPUTS
 }
 

@@ -89,7 +89,7 @@ def gated_delta(proj: torch.Tensor, a_off: int, b_off: int, conv: torch.Tensor, 
     gates = torch.empty((tokens, heads, 2), dtype=torch.float32, device=proj.device)
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=proj.device)
     coef = None
-    if by_groups:
+    if by_groups and most > 1:
         coef = torch.empty((tokens // 4 + step.sequences, heads,
                             plain_function("sakv_delta_coefficients")()),
                            dtype=torch.float32, device=proj.device)

@@ -88,7 +88,7 @@ class GatedDeltaMixer(Part):
         o = ops.gated_delta(mine, a_off, a_off + s.heads, self.conv_w, self.a, self.dt_bias,
                             conv_view.state, state_view.state, step, s.heads, s.kv_heads,
                             s.head_dim, s.value_dim, s.q_scale, s.unit_eps, keep_state=write_cache,
-                            by_groups=self.act_dtype != torch.float32 and step.max_new > 1)
+                            by_groups=self.act_dtype != torch.float32)
         return ops.norm_gate(o, self.norm_w, mine[:, g_off:a_off], s.eps, 1.0, self.act_dtype,
                              group=s.value_dim, gate_silu=True)
 
