@@ -33,6 +33,8 @@ class RoutedExperts(Part):
 
     def __init__(self, spec, prefix, mode):
         super().__init__(spec, prefix, mode)
+        if spec.shared is not None and mode == "bfloat16":
+            self.kernel_libraries += ("gemm_pair",)       # (the shared expert's gated product)
         if spec.score not in ("sigmoid", "softmax"):
             raise ValueError(f"router score {spec.score!r}: 'sigmoid' and 'softmax' are built")
         self.outputs = spec.experts + spec.identity
@@ -112,10 +114,9 @@ class RoutedExperts(Part):
         products = mixture.grouped_product(act, routing, self.w_down, None)
         shared = gate = None
         if s.shared is not None:
-            both = ops.linear(h, self.w_shared_in, out_dtype=self.act_dtype)
-            shared = ops.linear(mixture.clamped_act(both, s.shared.limit, s.shared.alpha,
-                                                    s.shared.plus),
-                                self.w_shared_down, out_dtype=torch.float32)
+            act = ops.gated_up(h, self.w_shared_in,
+                               (s.shared.limit, s.shared.alpha, s.shared.plus))
+            shared = ops.linear(act, self.w_shared_down, out_dtype=torch.float32)
             gate = logits[:, self.outputs] if self.has_gate else None
         return mixture.combine(products, routing, not s.weight_input, shared, gate, h, into)
 
