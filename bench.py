@@ -884,8 +884,8 @@ def gozolix_configs(size: dict) -> dict:
                 layers.append({"type": "attention", "mlp": m,
                                "mixer": own if i < 3 else dict(own, kv_from=2)})
         return {"architecture": "Gozolix", **common, "layers": layers,
-                "embedding": {"scale": 1.0, "bigram": {"buckets": 32749, "mul_prev": 31,
-                                                       "mul_cur": 7}}}
+                "embedding": {"scale": 1.0, "bigram": {"buckets": 32749, "mul_prev": 17,
+                                                       "mul_cur": 3}}}
 
     other, _ = design_configs(dict(size, delta=(dheads, ddim), streams=None, window=None,
                                    attention=(heads, kv_heads, dim)))

@@ -64,7 +64,7 @@ def draw(seed, all_chosen=False):
                                 temp, mlp(), source))
     embedding = {"scale": float(pick([1.0, 2.0, 5.0]))}
     if rng.random() < 0.8:
-        embedding["bigram"] = bigram(pick([1, 7, 97, 1000]), pick([1, 31, 1009]), pick([1, 7, 65537]))
+        embedding["bigram"] = bigram(pick([1, 7, 97, 1000]), pick([1, 29, 1009]), pick([1, 11, 65537]))
     return {"architecture": "Gozolix", "vocab": int(rng.integers(50, 700)), "width": width,
             "norm": {"eps": float(pick([1e-6, 1e-5]))}, "embedding": embedding,
             "initializer_range": 0.1, "layers": layers}
